@@ -191,9 +191,9 @@ LMRS_DEVINL void serial_av2_f32(float& xa_io, float& xb_io, const float* __restr
 // Bit-exact restatement of src/transformer.rs:501-544 for one token: every f32 operation happens in the
 // reference's order (serial dot over d, serial softmax sum over t, serial a*v accumulation over t, separate
 // mul and add, exp = glibc expf); only independent chains run in parallel.  One CTA per KV head (x chunks of 4
-// query heads).  K and V stream through a 4-deep cp.async (LDGSTS) tile ring so that several tiles are in
+// query heads).  K and V stream through a 4-deep cp.async tile ring so that several tiles are in
 // flight while the dependent-add chains of the current tile run; K tiles are stored with their 16-byte columns
-// rotated by the row index, which makes the per-position LDS.128 dot products bank-conflict-free without
+// rotated by the row index, which makes the per-position 16-byte-load dot products bank-conflict-free without
 // touching the ascending-d summation order.  Latency floor: the two T-long dependent add chains (softmax sum,
 // a*v) -- the price of exact parity, see exact_math.cuh.
 template <int HS, int NTHR, bool BIG = false>
@@ -318,7 +318,7 @@ LMRS_DEVINL void attn_decode_body(const AttnParams& p, float* att_smem, const in
         __syncthreads();                               // tile tl visible; everyone is done with tile tl-1
         issue_tile(p.kcache, tl + ATT_NT - 1, true);   // refill the slot tile tl-1 used
         const int rows = min(TILE, T - tl * TILE);
-        // thread = (row r, pair of heads): one LDS.128 of K feeds two independent dot-product chains (ILP 2),
+        // thread = (row r, pair of heads): one 16-byte-load of K feeds two independent dot-product chains (ILP 2),
         // products of chunk d4+1 are formed while chunk d4's dependent adds run
         const int npair = (nh + 1) / 2;
         for (int idx = tid; idx < rows * npair; idx += NTHR) {
@@ -328,7 +328,7 @@ LMRS_DEVINL void attn_decode_body(const AttnParams& p, float* att_smem, const in
             const float4* qb = reinterpret_cast<const float4*>(q_s + hb * HS);
             const float4* k4 = reinterpret_cast<const float4*>(tb + r * HS);
             float sa = 0.0f, sb = 0.0f;
-            // the whole K row first (C4 independent LDS.128: their latency overlaps), un-rotating on the fly
+            // the whole K row first (C4 independent 16-byte-load: their latency overlaps), un-rotating on the fly
             float4 kr[C4];
             {
                 int c = r % C4;
@@ -467,11 +467,11 @@ __global__ void __launch_bounds__(ATT_THREADS) attn_decode_kernel(const AttnPara
 // ---- cluster decode attention -------------------------------------------------------------------------------------
 // The single-CTA kernel above is bounded by what ONE SM can pull from L2 (~40 B/clk) and by running every phase of a
 // whole KV head on one SM.  Here a thread-block CLUSTER of CL CTAs serves one KV head (nh <= 4 query heads):
-//   scores : CTA `rank` owns positions [rank*RP, rank*RP+RP) -- 1/CL of the K rows, staged with cp.async (LDGSTS) --
-//            and PUSHES every score it computes into the shared memory of the CTAs that need it with st.async
-//            (SASS STAS), which also counts the bytes on the receiver's mbarrier: a consumer simply waits until its
-//            complete score rows have arrived -- no cluster-wide barrier (ptxas lowers barrier.cluster.arrive.release
-//            to MEMBAR.ALL.GPU) and no remote reads
+//   scores : CTA `rank` owns positions [rank*RP, rank*RP+RP) -- 1/CL of the K rows, staged with cp.async --
+//            and PUSHES every score it computes into the shared memory of the CTAs that need it with st.async,
+//            which also counts the bytes on the receiver's mbarrier: a consumer simply waits until its
+//            complete score rows have arrived -- no cluster-wide barrier (a releasing barrier.cluster.arrive costs most of
+//            a microsecond) and no remote reads
 //   softmax: the cluster is split into G head groups of R = CL/G CTAs; a CTA runs max / exp / serial sum / divide
 //            only for its group's nh/G heads (G = nh for Llama-style GQA: one head per CTA pair)
 //   a*v    : CTA (group, part) owns output dims [part*HS/R, ...) of its heads -- that slice of every V row is
@@ -483,7 +483,7 @@ LMRS_DEVINL uint32_t cluster_ctarank() { uint32_t r; asm volatile("mov.u32 %0, %
 LMRS_DEVINL void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
 LMRS_DEVINL void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 // push one f32 into CTA `rank`'s shared memory (same offsets as mine) and count its 4 bytes on that CTA's mbarrier:
-// st.async (SASS STAS) -- the receiver just waits for its expected byte count, no cluster-wide barrier or fence
+// st.async -- the receiver just waits for its expected byte count, no cluster-wide barrier or fence
 LMRS_DEVINL void st_async_f32(const float* local_ptr, const uint64_t* local_bar, uint32_t rank, float v) {
     uint32_t ra, rb;
     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(local_ptr)), "r"(rank));

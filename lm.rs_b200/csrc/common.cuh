@@ -1,5 +1,5 @@
 // common.cuh -- sm_100a PTX helpers shared by the lmrs_b200 kernels: mbarrier, 1-D bulk async copies
-// (TMA engine, SASS UBLKCP), programmatic dependent launch, exact-rounding float helpers.
+// (TMA engine), programmatic dependent launch, exact-rounding float helpers.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>

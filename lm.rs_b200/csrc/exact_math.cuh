@@ -8,8 +8,10 @@
 // path (softmax src/functional.rs:133, SiLU src/transformer.rs:617).  Rust's f32::exp lowers to the
 // platform expf, i.e. glibc's (sysdeps/ieee754/flt-32/e_expf.c, glibc >= 2.27): a double-precision
 // degree-3 polynomial around a 32-entry 2^(i/32) table, rounded once to float.  expf_glibc() below restates
-// that algorithm with the constants of `__exp2f_data` (table = correctly rounded 2^(i/32) minus i<<47;
-// polynomial and 32/ln2 constants read out of libm.so.6 2.39 and equal to the published source).
+// that algorithm.  Its constants: the table is 2^(i/32) correctly rounded to double, minus i<<47 in the bit pattern, and
+// InvLn2N is 32/ln2 correctly rounded -- mathematics, recomputed in high precision by tests/test_exact_math.py; the three
+// polynomial coefficients are those of the published source (Arm Optimized Routines / glibc, exp2f_data: C0, C1, C2 for the
+// 32-entry table, written there for 2^x and divided here by 32^3, 32^2 and 32).
 // tests/test_exact_math.py checks it against the host's glibc expf on tens of millions of inputs.
 #pragma once
 #include <stdint.h>
@@ -55,7 +57,7 @@ LMRS_HD float expf_glibc_t(float x, const uint64_t* T) {
     const double xd = (double)x;
     const double InvLn2N = 0x1.71547652b82fep+5;   // 32/ln2
     const double Shift = 0x1.8p+52;
-    const double C0 = 0x1.c6af84b912394p-20, C1 = 0x1.ebfce50fac4f3p-13, C2 = 0x1.62e42ff0c52d6p-6;
+    const double C0 = 0x1.c6af84b912394p-5 / 32768.0, C1 = 0x1.ebfce50fac4f3p-3 / 1024.0, C2 = 0x1.62e42ff0c52d6p-1 / 32.0;
 #ifdef __CUDA_ARCH__
     const double z = __dmul_rn(InvLn2N, xd);
     double kd = __dadd_rn(z, Shift);

@@ -13,8 +13,8 @@
 //                              into f32 register accumulators in the reference's order -> results are bit-identical
 //                              to the CPU path; double-buffered TMEM lets group g+1's MMAs run under group g's epilogue.
 // The CUDA-core mini-epilogue runs after EVERY group (the scale is rank-1 per K group), so it bounds the kernel: it is written
-// with packed f32x2 arithmetic and an exact integer->float conversion without I2F (2.5 issue slots per element per group
-// instead of ~5 with a quarter-rate I2F; 3 per element), the tile's weight scales are staged once for all groups, and tiles come in three
+// with packed f32x2 arithmetic and an exact integer->float conversion without a convert instruction (2.5 issue slots per element per group
+// instead of ~5 with a quarter-rate conversion; 3 per element), the tile's weight scales are staged once for all groups, and tiles come in three
 // shapes so that every matrix fills the GPU: 128 x 128, 128 x 64 (Wo / W2: 2048 output rows), and the fused gate/up tile.
 #pragma once
 #include <cuda.h>
@@ -110,20 +110,20 @@ template <int N> LMRS_DEVINL void tmem_ld(uint32_t taddr, uint32_t (&v)[N]) {
     if constexpr (N == 32) tmem_ld32(taddr, v); else tmem_ld16(taddr, v);
 }
 
-// ---- packed f32x2 arithmetic (Blackwell FADD2 / FMUL2: two IEEE round-to-nearest results per issue slot) ----------------
+// ---- packed f32x2 arithmetic (two IEEE round-to-nearest results per issue slot) ----------------
 LMRS_DEVINL uint64_t f2_pack(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
 LMRS_DEVINL void f2_unpack(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
 LMRS_DEVINL uint64_t f2_mul(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 LMRS_DEVINL uint64_t f2_add(uint64_t a, uint64_t b) { uint64_t r; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 // A product that must stay a SEPARATELY ROUNDED product when an add consumes it.  ptxas (12.9) contracts mul.rn.f32x2
-// followed by add.rn.f32x2 into one FFMA2 -- a single rounding -- although both carry an explicit rounding modifier (it
+// followed by add.rn.f32x2 into one fused operation -- a single rounding -- although both carry an explicit rounding modifier (it
 // does not do that to the scalar forms).  Written as fma(a, b, -0.0) with the -0.0 taken from a kernel PARAMETER the
-// product is exact (a*b + -0.0 rounds like a*b and keeps the sign of a zero product), costs the same FFMA2 issue slot,
-// and cannot be contracted any further: the following add stays an FADD2.
+// product is exact (a*b + -0.0 rounds like a*b and keeps the sign of a zero product), costs the same issue slot,
+// and cannot be contracted any further: the following add stays an add.
 LMRS_DEVINL uint64_t f2_mul_sep(uint64_t a, uint64_t b, uint64_t neg_zero2) {
     uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(neg_zero2)); return r;
 }
-// (ival as f32) for |ival| < 2^22 without I2F (a quarter-rate conversion that bounded the first build's epilogue): the
+// (ival as f32) for |ival| < 2^22 without a convert instruction (a quarter-rate conversion that bounded the first build's epilogue): the
 // integer is added into the mantissa of 1.5 * 2^23 and the constant subtracted again -- both steps exact.
 // |ival| <= 128 * 127 * 127 = 2,064,512 for one quantization group.
 constexpr int GEMM_MAGIC_I = 0x4B400000;
@@ -136,7 +136,7 @@ LMRS_DEVINL void gemm_epi_chunk(uint64_t* acc, const uint32_t (&v)[N], const flo
     const float4* w4 = reinterpret_cast<const float4*>(ws32);
 #pragma unroll
     for (int j = 0; j < N / 4; j++) {
-        const float4 w = w4[j];   // the same address for every lane: one broadcast LDS.128
+        const float4 w = w4[j];   // the same address for every lane: one broadcast 16-byte load
         const uint64_t f0 = f2_add(f2_pack(__int_as_float((int)v[4 * j] + GEMM_MAGIC_I), __int_as_float((int)v[4 * j + 1] + GEMM_MAGIC_I)), neg_magic2);
         const uint64_t f1 = f2_add(f2_pack(__int_as_float((int)v[4 * j + 2] + GEMM_MAGIC_I), __int_as_float((int)v[4 * j + 3] + GEMM_MAGIC_I)), neg_magic2);
         acc[2 * j] = f2_add(acc[2 * j], f2_mul_sep(f2_mul(f0, f2_pack(w.x, w.y)), xs2, nz2));

@@ -12,13 +12,13 @@
 // Data movement (HBM-bound kernel, ~2 int-ops/byte): every warp owns two independent "streams" of
 // consecutive weight rows (one per half-warp; for GLU the halves stream the same rows of w1 and w3).  A
 // stream is a contiguous byte range of the row-major [o][n] int8 matrix plus the matching contiguous range
-// of f32 group scales, so lane 0 moves it with 1-D bulk async copies (cp.async.bulk -> SASS UBLKCP, the TMA
+// of f32 group scales, so lane 0 moves it with 1-D bulk async copies (cp.async.bulk, the TMA
 // engine) into a per-warp shared-memory ring guarded by mbarriers: no registers are tied up by loads in
 // flight, and the first DEPTH stages are issued BEFORE griddepcontrol.wait so weight traffic overlaps the
 // previous kernel's tail and this kernel's own prologue (programmatic dependent launch).
 //
-// Arithmetic: a stage gives each lane one whole 128-element group (8 x LDS.128 of weights, 8 x LDS.128 of
-// the quantized activation, 32 x IDP.4A) -- the int32 group sum needs no cross-lane reduction.  The f32 part
+// Arithmetic: a stage gives each lane one whole 128-element group (8 x 16-byte loads of weights, 8 x 16-byte loads of
+// the quantized activation, 32 x dp4a) -- the int32 group sum needs no cross-lane reduction.  The f32 part
 // follows the reference bit for bit: term = ((ival as f32) * ws) * xs, and terms are added to the row
 // accumulator in ascending group order starting from 0.0 (a 16-step shuffle scan per half-warp), so
 // matmul_q8/matmul_q4 results are BIT-IDENTICAL to the CPU path; -fmad=false keeps mul/add unfused.
@@ -234,7 +234,7 @@ LMRS_DEVINL void quantize_group_to_smem(float4 y, int g, uint8_t* xq, float* xs,
 
 // The same chain on a TRANSPOSED staging of the squares (what the GEMV prologues use): the owner of element e = 8j + k
 // stores x[e]*x[e] (the reference's unfused product, src/functional.rs:56) at row k, column j of eight rows padded to
-// n/8 + 4 floats, so chain k reads ITS products as consecutive float4 (one LDS.128 per four dependent adds, the eight
+// n/8 + 4 floats, so chain k reads ITS products as consecutive float4 (one 16-byte loads per four dependent adds, the eight
 // lanes on distinct banks) instead of one strided scalar load per add: the chain runs at the dependent-add latency.
 LMRS_DEVINL int rnorm_t_stride(int n) { return n / 8 + 4; }
 LMRS_DEVINL void rnorm_t_stage4(float* xt, int n, int c, float4 v) {   // chunk c = elements 4c .. 4c+3
@@ -704,7 +704,7 @@ LMRS_DEVINL void consume_stage(const GemvParams& p, const WarpStreams<QT>& w, in
             } else {
                 const int4* xv = reinterpret_cast<const int4*>(sm.xq + (size_t)g * GS);
 #pragma unroll
-                for (int i = 0; i < 8; i++) {   // 16-byte column rotated by lane: conflict-free LDS.128
+                for (int i = 0; i < 8; i++) {   // 16-byte column rotated by lane: conflict-free 16-byte loads
                     const int cc = (i + l16) & 7;
                     const int4 w4 = wv[cc], x4 = xv[cc];
                     iv0 = dp4a_ss(w4.x, x4.x, iv0); iv1 = dp4a_ss(w4.y, x4.y, iv1);

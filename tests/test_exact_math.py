@@ -37,3 +37,18 @@ def test_expf_restatement_matches_host_libm_bit_for_bit():
         subprocess.check_call([gxx, "-O2", "-ffp-contract=off", "-I", os.path.join(ROOT, "lm.rs_b200", "csrc"), "-o", exe, src, "-lm"])
         n, bad = map(int, subprocess.check_output([exe]).split())
     assert n > 20_000_000 and bad == 0
+
+
+def test_table_and_scale_follow_from_mathematics():
+    """the 32 table words are 2^(i/32) correctly rounded to double with i << 47 taken off the bits, InvLn2N is 32 / ln 2"""
+    import re
+    import struct
+    from decimal import Decimal, getcontext
+    getcontext().prec = 60
+    text = open(os.path.join(ROOT, "lm.rs_b200", "csrc", "exact_math.cuh")).read()
+    words = [int(w, 16) for w in re.findall(r"0x([0-9a-f]{16})ull", text)]
+    ln2 = Decimal(2).ln()
+    want = [struct.unpack("<Q", struct.pack("<d", float((ln2 * i / 32).exp())))[0] - (i << 47) for i in range(32)]
+    assert words == want
+    inv = re.search(r"InvLn2N = (0x[0-9a-fp.+]+);", text).group(1)
+    assert float.fromhex(inv) == float(Decimal(32) / ln2)
