@@ -52,7 +52,7 @@ struct BdLayerCfg {
 template <typename AT, typename WT> class BadepelModel : public DenseModel<AT, WT> {
   public:
     typedef DenseModel<AT, WT> B;
-    using B::error; using B::launches; using B::info; using B::d_logits; using B::width; using B::vocab; using B::max_tokens;
+    using B::load_vec; using B::load_stack; using B::load_mat_f32; using B::error; using B::launches; using B::info; using B::d_logits; using B::width; using B::vocab; using B::max_tokens;
     using B::sms; using B::d_tokens; using B::cap; using B::x; using B::hn; using B::d_rows; using B::MAX_SPLIT; using B::pdl_now;
     using B::dalloc; using B::dfree; using B::need; using B::upload_w; using B::upload_f32; using B::check_launch; using B::launch_k;
     using B::drop_graphs; using B::optin;
@@ -156,28 +156,6 @@ template <typename AT, typename WT> class BadepelModel : public DenseModel<AT, W
     }
 
     // ---- weights -----------------------------------------------------------------------------------------------------------
-    int load_vec(const SafeTensors& st, const std::string& name, int n, float** out) {
-        const StTensor* t = nullptr;
-        return need(st, name, {n}, &t) || upload_f32(t, out);
-    }
-    int load_mat_f32(const SafeTensors& st, const std::string& name, int rows, int cols, float** out) {
-        const StTensor* t = nullptr;
-        return need(st, name, {rows, cols}, &t) || upload_f32(t, out);
-    }
-    // matrices stacked into one: rows of `parts` in order
-    int load_stack(const SafeTensors& st, const std::vector<std::pair<std::string, int>>& parts, int K, WT** out, int* rows_out) {
-        int rows = 0;
-        for (const auto& pr : parts) rows += pr.second;
-        if (dalloc(out, (size_t)rows * K)) return 1;
-        int r0 = 0;
-        for (const auto& pr : parts) {
-            const StTensor* t = nullptr;
-            if (need(st, pr.first, {pr.second, K}, &t) || upload_w(t, *out + (size_t)r0 * K)) return 1;
-            r0 += pr.second;
-        }
-        if (rows_out) *rows_out = rows;
-        return 0;
-    }
     // vectors ([n]) or tap tables ([n][inner]) laid end to end as f32, then `pad` zeros
     int load_f32_stack(const SafeTensors& st, const std::vector<std::pair<std::string, int>>& parts, int inner, int pad, float** out) {
         std::vector<float> host;

@@ -214,7 +214,10 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_const
                         const float bias = p.e.bias ? p.e.bias[o] : 0.0f;
 #pragma unroll 8
                         for (int r = 0; r < 32; r++)
-                            if (t0 + r < row_end) dst[(size_t)r * p.e.ldo] = p.e.bias ? stg[r * 33 + lane] * p.e.scale + bias : stg[r * 33 + lane] * p.e.scale;
+                            if (t0 + r < row_end) {
+                                const float a = p.e.bias ? stg[r * 33 + lane] * p.e.scale + bias : stg[r * 33 + lane] * p.e.scale;
+                                dst[(size_t)r * p.e.ldo] = p.e.softcap > 0.0f ? p.e.softcap * tanhf(a / p.e.softcap) : a;
+                            }
                     } else if constexpr (EPI == EPI_RESID) {
                         float* __restrict__ dst = p.e.out + (size_t)t0 * p.e.ldo + o;
                         const float lsv = p.e.ls[o], lbv = p.e.lb ? p.e.lb[o] : 0.0f;

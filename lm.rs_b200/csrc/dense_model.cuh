@@ -162,6 +162,31 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         return 0;
     }
 
+    int load_vec(const SafeTensors& st, const std::string& name, int n, float** out) {
+        const StTensor* t = nullptr;
+        return need(st, name, {n}, &t) || upload_f32(t, out);
+    }
+    int load_mat_f32(const SafeTensors& st, const std::string& name, int rows, int cols, float** out) {
+        const StTensor* t = nullptr;
+        return need(st, name, {rows, cols}, &t) || upload_f32(t, out);
+    }
+    // matrices stacked into one: rows of `parts` in order, then zero rows up to a multiple of `row_multiple`
+    int load_stack(const SafeTensors& st, const std::vector<std::pair<std::string, int>>& parts, int K, WT** out, int* rows_out, int row_multiple = 1) {
+        int rows = 0;
+        for (const auto& pr : parts) rows += pr.second;
+        const int padded = (rows + row_multiple - 1) / row_multiple * row_multiple;
+        if (dalloc(out, (size_t)padded * K)) return 1;
+        if (padded > rows) GCK(cudaMemset(*out + (size_t)rows * K, 0, (size_t)(padded - rows) * K * sizeof(WT)));
+        int r0 = 0;
+        for (const auto& pr : parts) {
+            const StTensor* t = nullptr;
+            if (need(st, pr.first, {pr.second, K}, &t) || upload_w(t, *out + (size_t)r0 * K)) return 1;
+            r0 += pr.second;
+        }
+        if (rows_out) *rows_out = padded;
+        return 0;
+    }
+
     // ---- launches -------------------------------------------------------------------------------------------------------
     int check_launch(const char* what) {
         launches++;
@@ -264,9 +289,9 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         gemm_tiled_kernel<AT, WT, EPI><<<dim3((O + 63) / 64, (std::min(T, max_group_rows) + 63) / 64, n_groups), 256, 0, st>>>(p);
         return check_launch("gemm_tiled_kernel");
     }
-    template <int EPI, int NORM> int launch_gemv(cudaStream_t st, GemvRowsParams<AT, WT> p, int nb = 1) {
+    template <int EPI, int NORM, int TAIL = TAIL_LAYER> int launch_gemv(cudaStream_t st, GemvRowsParams<AT, WT> p, int nb = 1) {
         const size_t smem = ((size_t)((p.K + 3) & ~3) + 36 + 2 * 8 + 4) * 4;
-        if (optin(gemv_rows_kernel<AT, WT, EPI, NORM>, smem)) return 1;
+        if (optin(gemv_rows_kernel<AT, WT, EPI, NORM, TAIL>, smem)) return 1;
         const int rows_per_cta = EPI == EPI_GLU ? 8 : 16;
         int grid = (p.O + rows_per_cta - 1) / rows_per_cta;
         // few rows: the warps of a CTA split K instead (two row pairs per CTA)
@@ -274,28 +299,28 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         if (p.ksplit) grid = (p.O + 3) / 4;
         p.pdl = pdl_now ? 1 : 0;
         grid = std::max(1, std::min(grid, sms * 4));
-        return launch_k("gemv_rows_kernel", st, pdl_now, gemv_rows_kernel<AT, WT, EPI, NORM>, dim3(grid, nb), dim3(256), smem, p);
+        return launch_k("gemv_rows_kernel", st, pdl_now, gemv_rows_kernel<AT, WT, EPI, NORM, TAIL>, dim3(grid, nb), dim3(256), smem, p);
     }
 
-    template <int RW, int NI> int launch_attn_t(cudaStream_t st, AttnRowsParams<AT> p, int grid_x, int grid_y) {
+    template <int RW, int NI, bool SIG> int launch_attn_t(cudaStream_t st, AttnRowsParams<AT> p, int grid_x, int grid_y) {
         // double-buffered K/V tiles when the head sizes allow 16-byte copies and two CTAs still fit an SM
         p.nbuf = (p.dk % 4 == 0 && p.dv % 4 == 0 && p.k_ld % 4 == 0 && p.v_ld % 4 == 0 && attn_smem_bytes<RW, NI>(p.dk, p.dv, 2) <= 100 * 1024) ? 2 : 1;
         const size_t smem = attn_smem_bytes<RW, NI>(p.dk, p.dv, p.nbuf);
-        if (optin(attn_rows_kernel<AT, RW, NI>, smem)) return 1;
-        return launch_k("attn_rows_kernel", st, pdl_now, attn_rows_kernel<AT, RW, NI>, dim3(grid_x, grid_y, p.nsplit), dim3(ATT_WARPS * 32), smem, p);
+        if (optin(attn_rows_kernel<AT, RW, NI, SIG>, smem)) return 1;
+        return launch_k("attn_rows_kernel", st, pdl_now, attn_rows_kernel<AT, RW, NI, SIG>, dim3(grid_x, grid_y, p.nsplit), dim3(ATT_WARPS * 32), smem, p);
     }
-    template <int RW> int launch_attn_rw(cudaStream_t st, const AttnRowsParams<AT>& p, int gx, int gy) {
+    template <int RW, bool SIG> int launch_attn_rw(cudaStream_t st, const AttnRowsParams<AT>& p, int gx, int gy) {
         const int ni = (p.dv + 31) / 32;
-        if (ni <= 1) return launch_attn_t<RW, 1>(st, p, gx, gy);
-        if (ni <= 2) return launch_attn_t<RW, 2>(st, p, gx, gy);
-        if (ni <= 4) return launch_attn_t<RW, 4>(st, p, gx, gy);
-        return launch_attn_t<RW, 8>(st, p, gx, gy);
+        if (ni <= 1) return launch_attn_t<RW, 1, SIG>(st, p, gx, gy);
+        if (ni <= 2) return launch_attn_t<RW, 2, SIG>(st, p, gx, gy);
+        if (ni <= 4) return launch_attn_t<RW, 4, SIG>(st, p, gx, gy);
+        return launch_attn_t<RW, 8, SIG>(st, p, gx, gy);
     }
     // attention over T query rows: the caller fills the tensors, head geometry, pitches, scale, soft-cap, window, kept first keys,
     // sink, gates and penalty;
     // the tiling, the key split of a one-row step and the merge of the splits are chosen here.  `part` is the split scratch
-    // [H][MAX_SPLIT][dv + 2].  A one-row step's launches depend on pos_hint only through its 64-position bucket.
-    int attention_launch(cudaStream_t st, AttnRowsParams<AT> p, float* part, uint32_t pos_hint) {
+    // [H][MAX_SPLIT][dv + 2].  SIG: independent sigmoid weights instead of the softmax.  A one-row step's launches depend on pos_hint only through its 64-position bucket.
+    template <bool SIG = false> int attention_launch(cudaStream_t st, AttnRowsParams<AT> p, float* part, uint32_t pos_hint) {
         const int kv_mul = p.H / p.G, T = p.T;
         p.part = part;
         if (p.out_ld == 0) p.out_ld = p.H * p.dv;
@@ -304,6 +329,7 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         int tiles = (int)((pos_hint + 1 + ATT_KT - 1) / ATT_KT);
         if (p.window > 0)   // tiles a window can touch, and those of the first keys that stay visible
             tiles = std::min(tiles, (p.window + ATT_KT - 2) / ATT_KT + 1 + (p.keep_first > 0 ? (p.keep_first + ATT_KT - 1) / ATT_KT : 0));
+        if (p.chunk > 0) tiles = std::min(tiles, (p.chunk + ATT_KT - 2) / ATT_KT + 1);
         tiles = std::min(tiles, MAX_SPLIT);
         // a one-row step over few KV heads: fewer query heads per CTA, so that more SMs share the keys
         while (T == 1 && p.HC > 4 && p.G * ((kv_mul + p.HC - 1) / p.HC) * tiles < sms) p.HC /= 2;
@@ -316,7 +342,7 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
             p.nsplit = std::max(1, std::min({tiles, MAX_SPLIT, (2 * sms) / std::max(1, p.G * chunks)}));
         }
         const int gx = (T + p.TQ - 1) / p.TQ, gy = p.G * chunks;
-        int rc = rw == 1 ? launch_attn_rw<1>(st, p, gx, gy) : (rw == 2 ? launch_attn_rw<2>(st, p, gx, gy) : launch_attn_rw<4>(st, p, gx, gy));
+        int rc = rw == 1 ? launch_attn_rw<1, SIG>(st, p, gx, gy) : (rw == 2 ? launch_attn_rw<2, SIG>(st, p, gx, gy) : launch_attn_rw<4, SIG>(st, p, gx, gy));
         if (rc) return rc;
         if (p.nsplit > 1) {
             AttnCombineParams<AT> cp{};

@@ -6,6 +6,9 @@
 //   tanhnorm_rows_kernel     tanh(alpha * x) * w + b per element (a norm without statistics), same gather and output
 //   layernorm_rows_kernel    (x - mean) / sqrt(var + eps) * w per row; the result is stored, or scaled per column and added
 //                            to the residual stream, and the row that comes out is also written in the operand type
+//   resnorm_rows_kernel      residual <- residual + rms(sublayer output) * w, then the next sublayer's RMS norm of it (or that
+//                            row's factor alone), optionally mixed with the previous token's normed row (token shift)
+//   norm_shift_rows_kernel   the token shift of many rows whose norm factors are known
 //   gemv_rows_kernel         one token row:  weights streamed once (HBM-bound), optional fused RMS-norm prologue,
 //                            epilogues: store*scale+bias | x += ls * f(acc) + lb | act(gate) * up | store in the operand
 //                            type; a batch dimension (per-head matrices, or experts picked by a device-side index list)
@@ -14,8 +17,9 @@
 //   qkv_post_kernel          per head: unit RMS norm of q/k or partial rotary, value mixing with an earlier layer's
 //                            values, sigmoid head gate, K/V rows written to the cache
 //   attn_rows_kernel         causal softmax attention with score scale and tanh soft-cap, optional sliding window (with
-//                            first positions that stay visible), logarithmic distance penalty, a learned per-head sink
-//                            in the softmax denominator, per-head or per-element sigmoid output gates, grouped query
+//                            first positions that stay visible) or fixed chunks of positions, logarithmic distance penalty, a
+//                            learned per-head sink in the softmax denominator, or independent sigmoid weights with a bias
+//                            per head instead of the softmax, per-head or per-element sigmoid output gates, grouped query
 //                            heads, query tile x KV head per CTA, K and V rows
 //                            with their own pitch (V may be a prefix of the K row: attention over a shared latent),
 //                            optional split over the keys (decode) + attn_combine_kernel
@@ -233,6 +237,118 @@ template <typename AT> __global__ void __launch_bounds__(256) layernorm_rows_ker
                       p.out_f ? p.out_f + (size_t)r * p.ld_f : nullptr, p.out_op ? p.out_op + (size_t)r * p.ldo : nullptr);
 }
 
+// ---- normed sublayer outputs into one residual stream, with the next norm behind -------------------------------------------
+// One row through a whole CTA: load(c) gives the sublayer's output; with wb
+//     x[c] <- x[c] + load(c) / sqrt(mean(load^2) + eps) * wb[c]
+// (without wb the row is x itself), then with w_next the next sublayer's input
+//     g[c] = x[c] / sqrt(mean(x^2) + eps) * w_next[c];      h[c] = g[c] + (before[c] - g[c]) * mu[c]        (mu: token shift)
+// where `before` is the previous token's g: read from prev (zeros when `fresh`, the first token of a sequence), which then takes
+// this token's g.  inv_out asks for the factor 1 / sqrt(mean(x^2) + eps) instead of h.  Rows up to SANDWICH_CACHE * blockDim.x
+// columns stay in registers; longer ones are loaded again.
+constexpr int SANDWICH_CACHE = 12;
+template <typename AT, typename F>
+DN_DEVINL void sandwich_row(F load, int n, float* x, const float* wb, float eps, float* red, const float* w_next, const float* mu, float* prev,
+                            bool fresh, AT* h, float* inv_out) {
+    const bool cached = n <= SANDWICH_CACHE * (int)blockDim.x;
+    float v[SANDWICH_CACHE];
+    float ss = 0.0f;
+    if (cached) {
+        float xv[SANDWICH_CACHE];
+#pragma unroll
+        for (int i = 0; i < SANDWICH_CACHE; i++) {
+            const int c = threadIdx.x + i * blockDim.x;
+            v[i] = c < n ? (wb ? load(c) : x[c]) : 0.0f;
+            xv[i] = c < n && wb ? x[c] : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < SANDWICH_CACHE; i++) ss = fmaf(v[i], v[i], ss);
+        if (wb) {
+            const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+            ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < SANDWICH_CACHE; i++) {
+                const int c = threadIdx.x + i * blockDim.x;
+                if (c < n) { v[i] = xv[i] + v[i] * inv * wb[c]; x[c] = v[i]; }
+                ss = fmaf(v[i], v[i], ss);
+            }
+        }
+    } else if (wb) {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = load(c); ss = fmaf(a, a, ss); }
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+        ss = 0.0f;
+        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = x[c] + load(c) * inv * wb[c]; x[c] = a; ss = fmaf(a, a, ss); }
+    } else {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
+    }
+    if (!w_next && !inv_out) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
+    if (inv_out) {
+        if (threadIdx.x == 0) *inv_out = inv;
+        return;
+    }
+    auto finish = [&](int c, float a) {
+        a = a * inv * w_next[c];
+        if (mu) {
+            const float before = fresh ? 0.0f : prev[c];
+            prev[c] = a;
+            a = a + (before - a) * mu[c];
+        }
+        from_f(h[c], a);
+    };
+    if (cached) {
+#pragma unroll
+        for (int i = 0; i < SANDWICH_CACHE; i++) {
+            const int c = threadIdx.x + i * blockDim.x;
+            if (c < n) finish(c, v[i]);
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) finish(c, x[c]);   // this thread stored it above
+    }
+}
+template <typename AT> struct ResNormRowsParams {
+    const float* y; int ldy; const float* wb;      // wb null: no sublayer output
+    float* x; int ldx; int n; float eps;
+    const float* w_next; AT* h; int ldh;           // or null
+    const float* mu; float* prev;                  // one row only: the shift here
+    float* inv_out;                                // [T]: many rows: the factors for norm_shift_rows_kernel
+    PosSrc ps;
+};
+template <typename AT> __global__ void __launch_bounds__(256) resnorm_rows_kernel(const ResNormRowsParams<AT> p) {
+    __shared__ float red[33];
+    pdl_launch();
+    pdl_wait();
+    const int r = blockIdx.x;
+    const float* y = p.wb ? p.y + (size_t)r * p.ldy : nullptr;
+    sandwich_row<AT>([&](int c) { return y[c]; }, p.n, p.x + (size_t)r * p.ldx, p.wb, p.eps, red, p.w_next, p.mu, p.prev, p.mu && pos_of(p.ps) == 0,
+                     p.h ? p.h + (size_t)r * p.ldh : nullptr, p.inv_out ? p.inv_out + r : nullptr);
+}
+// g_t = x_t * inv[t] * w;  h_t = g_t + (g_{t-1} - g_t) * mu.  Row -1 is prev_in (zeros for a step at position 0); the last row's g
+// goes to prev_out (another buffer: blocks of the grid still read prev_in).  A thread walks NORM_SHIFT_ROWS rows of one column.
+constexpr int NORM_SHIFT_ROWS = 8;
+template <typename AT> struct NormShiftRowsParams {
+    const float* x; int ldx; const float* inv; const float* w; const float* mu;
+    const float* prev_in; float* prev_out;
+    AT* h; int ldh; int T, n;
+    PosSrc ps;
+};
+template <typename AT> __global__ void __launch_bounds__(256) norm_shift_rows_kernel(const NormShiftRowsParams<AT> p) {
+    pdl_launch();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, t0 = blockIdx.y * NORM_SHIFT_ROWS;
+    if (c >= p.n) return;
+    const float w = p.w[c], mu = p.mu[c];
+    float g[NORM_SHIFT_ROWS + 1];
+    g[0] = t0 > 0 ? p.x[(size_t)(t0 - 1) * p.ldx + c] * p.inv[t0 - 1] * w : (pos_of(p.ps) > 0 ? p.prev_in[c] : 0.0f);
+#pragma unroll
+    for (int i = 0; i < NORM_SHIFT_ROWS; i++) g[i + 1] = t0 + i < p.T ? p.x[(size_t)(t0 + i) * p.ldx + c] * p.inv[t0 + i] * w : 0.0f;
+#pragma unroll
+    for (int i = 0; i < NORM_SHIFT_ROWS; i++)
+        if (t0 + i < p.T) {
+            from_f(p.h[(size_t)(t0 + i) * p.ldh + c], g[i + 1] + (g[i] - g[i + 1]) * mu);
+            if (t0 + i == p.T - 1) p.prev_out[c] = g[i + 1];
+        }
+}
+
 // ---- several residual streams -------------------------------------------------------------------------------------------
 // Instead of one residual row a token carries S of them, X[0 .. S) (all equal to the embedding row at the start).  A sublayer
 // reads u = sum_s win[s] X[s] (then normalised), and its output y is written to every stream at once from the old ones:
@@ -374,6 +490,7 @@ template <typename AT> struct EpiParams {
     int glu_kind;             // EPI_GLU: GLU_SILU silu(gate) * up | GLU_CLAMPED g = min(gate, limit), u = clamp(up, +-limit):
     float glu_limit, glu_alpha;   //      g * sigmoid(glu_alpha * g) * (u + 1)
     int act_kind;             // EPI_ACT: ACT_NONE acc | ACT_RELU2 max(acc, 0)^2
+    float softcap;            // EPI_STORE: > 0: out = softcap * tanh(out / softcap) (capped logits)
 };
 enum { GLU_SILU = 0, GLU_CLAMPED = 1 };
 enum { ACT_NONE = 0, ACT_RELU2 = 1 };
@@ -390,7 +507,10 @@ template <typename AT> DN_DEVINL float act_apply(const EpiParams<AT>& e, float a
     return a;
 }
 template <int EPI, typename AT> DN_DEVINL void epi_apply(const EpiParams<AT>& e, int t, int o, float a, float b) {
-    if (EPI == EPI_STORE) e.out[(size_t)t * e.ldo + o] = e.bias ? a * e.scale + e.bias[o] : a * e.scale;
+    if (EPI == EPI_STORE) {
+        a = e.bias ? a * e.scale + e.bias[o] : a * e.scale;
+        e.out[(size_t)t * e.ldo + o] = e.softcap > 0.0f ? e.softcap * tanhf(a / e.softcap) : a;
+    }
     else if (EPI == EPI_RESID) {
         if (e.tanh_alpha) a = tanhf(*e.tanh_alpha * a);
         e.out[(size_t)t * e.ldo + o] += e.lb ? e.ls[o] * a + e.lb[o] : e.ls[o] * a;
@@ -413,10 +533,14 @@ enum { NORM_NONE = 0, NORM_RMS = 1, NORM_TANH = 2, NORM_LAYER = 3 };
 // -- every CTA takes a ticket from *counter after its stores -- sends the row e.out[0 .. O) through a layer norm into the
 // residual stream, x <- x + ls * LN(row) w, and writes x again in the operand type to h.  Nobody waits for anybody: the last
 // ticket simply falls to whoever comes last, and that CTA puts the counter back to zero.
+// The RMS form (kernels instantiated with TAIL_RMS) sends the row through sandwich_row instead: x <- x + rms(row) w, and the next
+// sublayer's input rms(x) w_next, token-shifted when mu is given, to h.
+enum { TAIL_LAYER = 0, TAIL_RMS = 1 };
 template <typename AT> struct LnTail {
     unsigned int* counter;
     const float* w; const float* ls; float eps;
     float* x; AT* h;
+    const float* w_next; const float* mu; float* prev; PosSrc ps;   // RMS form
 };
 template <typename AT, typename WT> struct GemvRowsParams {
     const AT* a;              // [K] input row (NORM_NONE)
@@ -496,7 +620,7 @@ DN_DEVINL void dot_rows(const WT* const (&w)[NR], const float* __restrict__ xs, 
 #pragma unroll
     for (int r = 0; r < NR; r++) out[r] = warp_sum(acc[r]);
 }
-template <typename AT, typename WT, int EPI, int NORM>
+template <typename AT, typename WT, int EPI, int NORM, int TAIL = TAIL_LAYER>
 static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsParams<AT, WT> pp) {
     extern __shared__ __align__(16) float gv_xs[];   // [K rounded up to 4] the input row as f32, then reduction slots
     GemvRowsParams<AT, WT> p = pp;
@@ -603,7 +727,11 @@ static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsPar
         if (last) {
             __threadfence();
             const float* row = p.e.out;
-            layernorm_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.w, p.ln.eps, red, p.ln.x, p.ln.ls, nullptr, p.ln.h);
+            if (TAIL == TAIL_RMS)
+                sandwich_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.x, p.ln.w, p.ln.eps, red, p.ln.w_next, p.ln.mu, p.ln.prev,
+                                 p.ln.mu && pos_of(p.ln.ps) == 0, p.ln.h, nullptr);
+            else
+                layernorm_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.w, p.ln.eps, red, p.ln.x, p.ln.ls, nullptr, p.ln.h);
             if (threadIdx.x == 0) *p.ln.counter = 0u;
         }
     }
@@ -703,6 +831,7 @@ struct QkvPostParams {
     int rot_dims; const float* rot_cos; const float* rot_sin;   // [max_tokens][rot_dims/2]
     int v_mode; float* v_first; const float* lambda;            // v_first [T][G*dv]; lambda: one float on the device
     bool has_gate;
+    bool q_only;              // no k and v columns: [q | gate logits] (a layer that reads another layer's cache)
     float* q_out; float* gate_out;
     float* kcache; float* vcache;                               // [max_tokens][G*dk], [max_tokens][G*dv]
     PosSrc ps;
@@ -717,7 +846,7 @@ static __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParam
     const int lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     const int wid = blockIdx.y * nw + (threadIdx.x >> 5), wtotal = gridDim.y * nw;
     const float* row = p.qkv + (size_t)t * p.ld;
-    const int n_qk = p.H + p.G, nv = p.G * p.dv, v_tasks = (nv + 127) / 128;
+    const int n_qk = p.q_only ? p.H : p.H + p.G, nv = p.q_only ? 0 : p.G * p.dv, v_tasks = (nv + 127) / 128;
     const float* vsrc = row + (size_t)n_qk * p.dk;
     const int n_tasks = n_qk + v_tasks + (p.has_gate ? 1 : 0);
     for (int task = wid; task < n_tasks; task += wtotal) {
@@ -769,7 +898,7 @@ static __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParam
 }
 
 // ---- attention --------------------------------------------------------------------------------------------------------
-// score = (q . k) * scale, then softcap * tanh(score / softcap) when softcap > 0, then minus r1[head] * ln(1 + r2[head] *
+// score = (q . k) * scale (SIG: see below), then softcap * tanh(score / softcap) when softcap > 0, then minus r1[head] * ln(1 + r2[head] *
 // distance) when r1 is given; row (t, head) at position i = pos+t sees keys j <= i, and only those with i - j < window or
 // j < keep_first when window > 0 (key tiles wholly between the kept first keys and the window are never loaded); softmax in
 // f32, its denominator enlarged by exp(sink[head]) when a sink is given; output row times the head's gate or times
@@ -786,6 +915,7 @@ constexpr int ATT_KT = 64, ATT_WARPS = 4;
 // cap * (1 - 2 / (e^(2s/cap) + 1)) then carries an absolute error of about cap * 1e-7 -- the size of the f32 rounding of the
 // score itself (a relative error near zero does not matter: what enters the softmax is the score's absolute value)
 DN_DEVINL float att_exp(float x) { return __expf(x); }
+DN_DEVINL float att_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }   // (a quotient by infinity is zero)
 DN_DEVINL float att_softcap(float s, float cap, float inv_cap2) {   // inv_cap2 = 2 / cap
     return cap * (1.0f - __fdividef(2.0f, __expf(s * inv_cap2) + 1.0f));
 }
@@ -799,6 +929,8 @@ template <typename AT> struct AttnRowsParams {
     int k_ld, v_ld;           // floats between consecutive positions of the K and of the V cache (>= G*dk, G*dv)
     int window;               // > 0: sliding window of that many keys (the row's own included); 0: all earlier keys
     int keep_first;           // with a window: keys at positions < keep_first stay visible to every later row
+    int chunk;                // > 0: row i sees key j only when both lie in the same block of `chunk` positions (counted from 0)
+    const float* wbias;       // sigmoid form: [H], added to the scaled score
     const float* sink;        // [H] or null: exp(sink[head]) is added to the softmax denominator (no key, no value, not scaled)
     const float* gate_logits; int gate_ld;   // or null: output element (t, h, c) is multiplied by sigmoid(gate_logits[t*gate_ld + h*dv + c])
     const float* r1; const float* r2;   // [H] distance penalty r1 * ln(1 + r2 * (i - j)), or null
@@ -819,7 +951,9 @@ template <int RW, int NI> inline size_t attn_smem_bytes(int dk, int dv, int nbuf
     const int d4 = (dk + 3) & ~3, R = RW * ATT_WARPS;
     return ((size_t)R * d4 + (size_t)nbuf * ((size_t)ATT_KT * attn_k_stride(dk) + (size_t)ATT_KT * 32 * NI) + (size_t)R * ATT_KT) * 4;
 }
-template <typename AT, int RW, int NI>
+// SIG: the weight of a visible key is sigmoid(score * scale + wbias[head]) and the weights are not normalised: no running maximum,
+// no rescaling, the denominator is one (soft-cap, sink and penalty do not apply)
+template <typename AT, int RW, int NI, bool SIG = false>
 static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const AttnRowsParams<AT> p) {
     constexpr int R = RW * ATT_WARPS, DVP = 32 * NI;
     pdl_launch();
@@ -858,7 +992,8 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
     const int n_keys = (int)pos0 + t_last + 1;           // keys this CTA's last row sees
     const int n_tiles = (n_keys + ATT_KT - 1) / ATT_KT;
     // the CTA's first row has the earliest window: tiles before its first visible key are skipped by every row
-    const int first_tile = p.window > 0 ? max(0, (int)pos0 + t0 - p.window + 1) / ATT_KT : 0;
+    const int first_tile = p.window > 0 ? max(0, (int)pos0 + t0 - p.window + 1) / ATT_KT
+                           : p.chunk > 0 ? ((int)pos0 + t0) / p.chunk * p.chunk / ATT_KT : 0;
     // ... except the tiles of the kept first keys: the walk is tiles 0 .. kf_tiles, then first_tile .. n_tiles
     const int kf_tiles = p.window > 0 && p.keep_first > 0 ? min(first_tile, (p.keep_first + ATT_KT - 1) / ATT_KT) : 0;
     const int n_walk = kf_tiles + n_tiles - first_tile;
@@ -872,6 +1007,7 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
         // the sink enters like a key with score sink[head] and no value; with split keys it belongs to split 0
         const bool sk = p.sink && r_ok[i] && blockIdx.z == 0;
         m[i] = sk ? p.sink[r_h[i]] : -1e30f; l[i] = sk ? 1.0f : 0.0f;
+        if (SIG) { m[i] = 0.0f; l[i] = split == 0 ? 1.0f : 0.0f; pen1[i] = r_ok[i] ? p.wbias[r_h[i]] : 0.0f; }
 #pragma unroll
         for (int c = 0; c < NI; c++) acc[i][c] = 0.0f;
     }
@@ -965,14 +1101,22 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
         for (int i = 0; i < RW; i++) {
             const int last = (int)pos0 + r_t[i];   // last visible key of this row
             float a = s0[i] * p.scale, b = s1[i] * p.scale;
+            if (SIG) {
+                const int first = p.chunk > 0 ? last / p.chunk * p.chunk : 0;   // first visible key
+                const int ja = j0 + lane, jb = ja + 32;
+                Ps[(size_t)(warp * RW + i) * ATT_KT + lane] = r_ok[i] && ja <= last && ja >= first ? att_sigmoid(a + pen1[i]) : 0.0f;
+                Ps[(size_t)(warp * RW + i) * ATT_KT + lane + 32] = r_ok[i] && jb <= last && jb >= first ? att_sigmoid(b + pen1[i]) : 0.0f;
+                continue;
+            }
             if (p.softcap > 0.0f) { a = att_softcap(a, p.softcap, inv_cap2); b = att_softcap(b, p.softcap, inv_cap2); }
             const int da = last - (j0 + lane), db = da - 32;   // distances of the two keys
             if (p.r1) {
                 a -= pen1[i] * __logf(1.0f + pen2[i] * (float)max(da, 0));
                 b -= pen1[i] * __logf(1.0f + pen2[i] * (float)max(db, 0));
             }
-            const bool va = r_ok[i] && da >= 0 && (p.window <= 0 || da < p.window || j0 + lane < p.keep_first);
-            const bool vb = r_ok[i] && db >= 0 && (p.window <= 0 || db < p.window || j0 + lane + 32 < p.keep_first);
+            const int first = p.chunk > 0 ? last / p.chunk * p.chunk : 0;
+            const bool va = r_ok[i] && da >= 0 && j0 + lane >= first && (p.window <= 0 || da < p.window || j0 + lane < p.keep_first);
+            const bool vb = r_ok[i] && db >= 0 && j0 + lane + 32 >= first && (p.window <= 0 || db < p.window || j0 + lane + 32 < p.keep_first);
             a = va ? a : -1e30f; b = vb ? b : -1e30f;
             const float mt = warp_max(fmaxf(a, b));
             const float mn = fmaxf(m[i], mt);
@@ -984,10 +1128,12 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
             Ps[(size_t)(warp * RW + i) * ATT_KT + lane + 32] = pb;
         }
         __syncwarp();
+        if (!SIG) {
 #pragma unroll
         for (int i = 0; i < RW; i++)
 #pragma unroll
             for (int c = 0; c < NI; c++) acc[i][c] *= corr[i];
+        }
         for (int j = 0; j < ATT_KT; j += 4) {
             float vv[4][NI];
 #pragma unroll
@@ -1067,6 +1213,7 @@ template <typename AT> struct CastColsParams {
     const float* in; int ld;
     AT* out; int ldo;
     int n, total;   // total = T * n
+    int tanh_first; // 1: the entry passes tanh on the way
 };
 template <typename AT> __global__ void __launch_bounds__(256) cast_cols_kernel(const CastColsParams<AT> p) {
     pdl_launch();
@@ -1074,7 +1221,8 @@ template <typename AT> __global__ void __launch_bounds__(256) cast_cols_kernel(c
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= p.total) return;
     const int t = i / p.n, c = i - t * p.n;
-    from_f(p.out[(size_t)t * p.ldo + c], p.in[(size_t)t * p.ld + c]);
+    const float v = p.in[(size_t)t * p.ld + c];
+    from_f(p.out[(size_t)t * p.ldo + c], p.tanh_first ? tanhf(v) : v);
 }
 
 // f32 <- bf16 widening of a weight tensor (the f32 operand mode keeps its weights as f32 in HBM)

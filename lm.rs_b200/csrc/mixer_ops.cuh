@@ -15,7 +15,11 @@
 //   delta_scan_kernel         S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q, token after token, the
 //                             state matrix of a head spread over the registers of the threads that own its columns; with one
 //                             decay per head instead of per key channel; or without the correction (gated linear attention:
-//                             S <- diag(g) S + k v^T)
+//                             S <- diag(g) S + k v^T); or with a decay and a removal rate per key channel (generalized delta
+//                             rule: S <- diag(w) S - (a u)(u^T S) + k v^T, u the unit key, both terms from the old S)
+//   general_delta_pre_kernel  what that last form needs per token and key channel: decays, removal vectors, the query's product
+//                             with the removal vector
+//   general_delta_step_kernel one token of it, from the projected row to the gated output row: decays, update, read-out, norm, gate
 //   gated_headnorm_kernel     o / rms(o) * w * sigmoid(gate) per head, in the operand type
 //   ssm_pre_kernel            state-space recurrence with one decay per head: short causal convolution + bias + SiLU over the
 //                             (x, B, C) channels, step sizes dt = softplus(raw + bias) and decays exp(-exp(A_log) dt)
@@ -347,11 +351,15 @@ struct DeltaScanParams {
     int T, H, G, dk, dv;
     PosSrc ps;
     float q_scale;              // the read-out times this constant (0: none)
+    const float* rem;           // SCAN_GENERAL: [T][H*dk] removal vectors
 };
 // what the scan computes per token.  SCAN_DELTA: the rule above with a decay per key channel.  SCAN_DELTA_HEAD: the same with
 // one decay per head (decay is [T][H]).  SCAN_PLAIN: no correction and no write strength, S <- diag(g) S + k v^T, o = S^T q
-// (gated linear attention): one pass over the registers and one lane reduction per token.
-enum { SCAN_DELTA = 0, SCAN_DELTA_HEAD = 1, SCAN_PLAIN = 2 };
+// (gated linear attention): one pass over the registers and one lane reduction per token.  SCAN_GENERAL: with a removal vector
+// b per token (rem; general_delta_pre_kernel folds the unit key's length into it) and s = S^T k from the OLD state,
+// S <- diag(g) S + k v^T - b s^T.  Nothing but that last subtraction waits for s: M = diag(g) S + k v^T and M^T q are formed
+// while s is being reduced, and o = M^T q - (q . b) s with the scalar q . b given in beta -- one round of lane reductions per token.
+enum { SCAN_DELTA = 0, SCAN_DELTA_HEAD = 1, SCAN_PLAIN = 2, SCAN_GENERAL = 3 };
 // (rows per lane NR, lanes per column LPC) for a key size: NR * LPC >= dk.  A warp issues dependent instructions only every few
 // cycles, so the split favours many lanes per column (more warps per scheduler, shorter chains) over few
 inline void delta_scan_shape(int dk, int* nr, int* lpc) {
@@ -362,7 +370,7 @@ inline void delta_scan_shape(int dk, int* nr, int* lpc) {
     else if (dk <= 256) { *nr = 8; *lpc = 32; }
     else { *nr = 16; *lpc = 32; }
 }
-inline size_t delta_scan_smem(int nr, int lpc) { return (size_t)2 * DELTA_TB * (3 * nr * lpc + DELTA_THREADS / lpc + 4) * 4; }
+inline size_t delta_scan_smem(int nr, int lpc, int mode = SCAN_DELTA) { return (size_t)2 * DELTA_TB * ((mode == SCAN_GENERAL ? 4 : 3) * nr * lpc + DELTA_THREADS / lpc + 4) * 4; }
 DN_DEVINL void cp_async4_zfill(void* smem_dst, const void* gsrc, bool valid) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
     const int n = valid ? 4 : 0;
@@ -373,7 +381,8 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
     pdl_launch();
     pdl_wait();
     constexpr int cols = DELTA_THREADS / LPC, dkp = NR * LPC;   // dkp: rows the lanes cover (>= dk, a multiple of 4)
-    constexpr int blk = DELTA_TB * (3 * dkp + cols + 4);                   // floats per staging buffer
+    constexpr int NA = MODE == SCAN_GENERAL ? 4 : 3;            // staged vectors of dkp entries per token: q, k, decays [, removal]
+    constexpr int blk = DELTA_TB * (NA * dkp + cols + 4);       // floats per staging buffer
     const int h = blockIdx.y, g = h / (p.H / p.G);
     const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC, j = blockIdx.x * cols + jl;
     const bool col_ok = j < p.dv;
@@ -381,12 +390,12 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
     const int vq = 2 * p.G * p.dk;
     // 16-byte copies when every row piece starts on a 16-byte boundary
     const bool vec = (p.dk & 3) == 0 && (p.ld & 3) == 0 && ((p.H * p.dk) & 3) == 0 && (reinterpret_cast<uintptr_t>(p.qkv) & 15) == 0 &&
-                     (reinterpret_cast<uintptr_t>(p.decay) & 15) == 0;
+                     (reinterpret_cast<uintptr_t>(p.decay) & 15) == 0 && (MODE != SCAN_GENERAL || (reinterpret_cast<uintptr_t>(p.rem) & 15) == 0);
     auto stage = [&](int t0, int buf) {
         float* qs = ds_sm + (size_t)buf * blk;     // [TB][dkp]
         float* ks = qs + DELTA_TB * dkp;
         float* gs = ks + DELTA_TB * dkp;
-        float* vs = gs + DELTA_TB * dkp;           // [TB][cols]
+        float* vs = qs + NA * DELTA_TB * dkp;      // [TB][cols]
         float* bs = vs + DELTA_TB * cols;          // [TB]
         const int nt = min(DELTA_TB, p.T - t0);
         if (vec) {
@@ -398,6 +407,7 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
                 cp_async16_zfill(qs + tt * dkp + i, ok ? row + g * p.dk + i : p.qkv, ok);
                 cp_async16_zfill(ks + tt * dkp + i, ok ? row + (p.G + g) * p.dk + i : p.qkv, ok);
                 if (MODE != SCAN_DELTA_HEAD) cp_async16_zfill(gs + tt * dkp + i, ok ? p.decay + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
+                if (MODE == SCAN_GENERAL) cp_async16_zfill(gs + (DELTA_TB + tt) * dkp + i, ok ? p.rem + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
             }
         } else {
             for (int e = threadIdx.x; e < nt * dkp; e += blockDim.x) {
@@ -407,6 +417,7 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
                 cp_async4_zfill(qs + tt * dkp + i, ok ? row + g * p.dk + i : p.qkv, ok);
                 cp_async4_zfill(ks + tt * dkp + i, ok ? row + (p.G + g) * p.dk + i : p.qkv, ok);
                 if (MODE != SCAN_DELTA_HEAD) cp_async4_zfill(gs + tt * dkp + i, ok ? p.decay + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
+                if (MODE == SCAN_GENERAL) cp_async4_zfill(gs + (DELTA_TB + tt) * dkp + i, ok ? p.rem + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
             }
         }
         for (int e = threadIdx.x; e < nt * cols; e += blockDim.x) {
@@ -434,10 +445,42 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
         const float* qs = ds_sm + (size_t)buf * blk;
         const float* ks = qs + DELTA_TB * dkp;
         const float* gs = ks + DELTA_TB * dkp;
-        const float* vs = gs + DELTA_TB * dkp;
+        const float* vs = qs + NA * DELTA_TB * dkp;
         const float* bs = vs + DELTA_TB * cols;
         for (int tt = 0; tt < nt; tt++) {
             float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
+            if (MODE == SCAN_GENERAL) {
+                const float* es = gs + DELTA_TB * dkp;   // removal vectors
+                const float v = vs[tt * cols + jl];
+                float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
+#pragma unroll
+                for (int r4 = 0; r4 < NR / 4; r4++) {
+                    const int i = (r4 * LPC + s) * 4;
+                    const float4 k4 = *reinterpret_cast<const float4*>(ks + tt * dkp + i);
+                    const float4 g4 = *reinterpret_cast<const float4*>(gs + tt * dkp + i);
+                    const float4 q4 = *reinterpret_cast<const float4*>(qs + tt * dkp + i);
+                    r0 = fmaf(S[4 * r4], k4.x, r0); r1 = fmaf(S[4 * r4 + 1], k4.y, r1);
+                    r2 = fmaf(S[4 * r4 + 2], k4.z, r2); r3 = fmaf(S[4 * r4 + 3], k4.w, r3);
+                    S[4 * r4] = fmaf(S[4 * r4], g4.x, k4.x * v); S[4 * r4 + 1] = fmaf(S[4 * r4 + 1], g4.y, k4.y * v);
+                    S[4 * r4 + 2] = fmaf(S[4 * r4 + 2], g4.z, k4.z * v); S[4 * r4 + 3] = fmaf(S[4 * r4 + 3], g4.w, k4.w * v);
+                    o0 = fmaf(S[4 * r4], q4.x, o0); o1 = fmaf(S[4 * r4 + 1], q4.y, o1);
+                    o2 = fmaf(S[4 * r4 + 2], q4.z, o2); o3 = fmaf(S[4 * r4 + 3], q4.w, o3);
+                }
+                float held = (r0 + r1) + (r2 + r3), om = (o0 + o1) + (o2 + o3);
+#pragma unroll
+                for (int o = LPC >> 1; o > 0; o >>= 1) {
+                    held += __shfl_xor_sync(0xffffffffu, held, o);
+                    om += __shfl_xor_sync(0xffffffffu, om, o);
+                }
+#pragma unroll
+                for (int r4 = 0; r4 < NR / 4; r4++) {
+                    const float4 e4 = *reinterpret_cast<const float4*>(es + tt * dkp + (r4 * LPC + s) * 4);
+                    S[4 * r4] = fmaf(-held, e4.x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held, e4.y, S[4 * r4 + 1]);
+                    S[4 * r4 + 2] = fmaf(-held, e4.z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held, e4.w, S[4 * r4 + 3]);
+                }
+                if (s == 0 && col_ok) p.out[(size_t)(t0 + tt) * p.H * p.dv + (size_t)h * p.dv + j] = fmaf(-held, bs[tt], om);
+                continue;
+            }
             if (MODE == SCAN_PLAIN) {
                 const float u = vs[tt * cols + jl];
 #pragma unroll
@@ -493,6 +536,144 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
     }
 }
 
+// ---- generalized delta rule ---------------------------------------------------------------------------------------------------
+// The projected row is [r (H*d) | k (H*d) | v (H*d) | gate logits (H*d) | removal logits (H*d) | decay latent]; z holds the decay
+// logits (second half of the low-rank projection, bias added).  Per token, head and key channel
+//     decay = exp(-decay_rate * sigmoid(z))          removal rate a = sigmoid(removal logit + bias)
+// and with u = k / sqrt(sum k^2 + 1e-6) the state update S <- diag(decay) S - (a u)(u^T S) + k v^T is what delta_scan_kernel's
+// SCAN_GENERAL does with b = a k / (sum k^2 + 1e-6) as the removal vector and s = S^T k.  Also the scalar r . b.  One warp per
+// (token, head); decays replace the logits in place.
+DN_DEVINL float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
+DN_DEVINL float general_decay(float z, float rate) { return expf(-rate * sigmoidf(z)); }
+struct GeneralDeltaPreParams {
+    const float* proj; int ld;
+    float* z;                  // [T][H*d] decay logits in, decays out
+    const float* a_bias;       // [H*d]
+    float* rem; float* rb;     // [T][H*d], [T][H]
+    int T, H, d;
+    float decay_rate;
+};
+static __global__ void __launch_bounds__(128) general_delta_pre_kernel(const GeneralDeltaPreParams p) {
+    pdl_launch();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (id >= p.T * p.H) return;
+    const int t = id / p.H, h = id - t * p.H, n = p.H * p.d;
+    const float* row = p.proj + (size_t)t * p.ld + (size_t)h * p.d;
+    float ss = 0.0f;
+    for (int i = lane; i < p.d; i += 32) { const float k = row[n + i]; ss += k * k; }
+    const float inv2 = 1.0f / (warp_sum(ss) + 1e-6f);
+    float rb = 0.0f;
+    const size_t o = (size_t)t * n + (size_t)h * p.d;
+    for (int i = lane; i < p.d; i += 32) {
+        const float b = sigmoidf(row[4 * n + i] + p.a_bias[(size_t)h * p.d + i]) * row[n + i] * inv2;
+        rb = fmaf(row[i], b, rb);
+        p.rem[o + i] = b;
+        p.z[o + i] = general_decay(p.z[o + i], p.decay_rate);
+    }
+    rb = warp_sum(rb);
+    if (lane == 0) p.rb[(size_t)t * p.H + h] = rb;
+}
+
+// One token of the rule, one CTA per head: the projected row in, the operand-type row rms(o) * w * sigmoid(gate) out.  The low-rank
+// latent passes tanh and is rounded to the operand type (what the many-token path feeds its product), the second half of the
+// projection is done here.  Threads are columns x row groups; the state goes past twice (once for S^T k, once for the update and
+// the read-out), the second time from L1.  Shared memory: ra + 4 d + blockDim.x floats (+ the reduction slots).
+template <typename AT, typename WT> struct GeneralDeltaStepParams {
+    const float* proj;         // the token's row; decay latent (before tanh) at column 5 * H * d
+    const WT* w2; int ra;      // [H*d][ra]
+    const float* w0; const float* a_bias; const float* w; float eps;
+    float* state;              // [H][d][d]
+    AT* out;                   // [H*d]
+    int H, d, cw;              // cw: columns per pass, a multiple of 32 that divides blockDim.x
+    float decay_rate;
+    PosSrc ps;
+};
+template <typename AT, typename WT> __global__ void __launch_bounds__(1024) general_delta_step_kernel(const GeneralDeltaStepParams<AT, WT> p) {
+    extern __shared__ __align__(16) float gd_sm[];
+    __shared__ float red[33];
+    pdl_launch();
+    pdl_wait();
+    const int h = blockIdx.x, d = p.d, n = p.H * d;
+    float* lat = gd_sm;            // [ra]
+    float* ks = lat + p.ra;        // [d] key
+    float* ws = ks + d;            // [d] decays
+    float* bs = ws + d;            // [d] removal vector
+    float* os = bs + d;            // [d] read-out
+    float* part = os + d;          // [blockDim.x] sums of the row groups
+    const float* row = p.proj + (size_t)h * d;
+    for (int i = threadIdx.x; i < p.ra; i += blockDim.x) { AT v; from_f(v, tanhf(p.proj[5 * (size_t)n + i])); lat[i] = to_f(v); }
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) { const float k = row[n + i]; ks[i] = k; ss += k * k; }
+    const float inv2 = 1.0f / (block_sum(ss, red) + 1e-6f);   // (its barriers also publish lat and ks)
+    // decay logits: eight lanes per key channel
+    for (int i0 = 0; i0 < d; i0 += blockDim.x >> 3) {
+        const int i = i0 + (threadIdx.x >> 3), l8 = threadIdx.x & 7;
+        float z = 0.0f;
+        if (i < d) {
+            const WT* w2 = p.w2 + ((size_t)h * d + i) * p.ra;
+            for (int j = l8; j < p.ra; j += 8) z = fmaf(to_f(w2[j]), lat[j], z);
+        }
+        z += __shfl_xor_sync(0xffffffffu, z, 4);
+        z += __shfl_xor_sync(0xffffffffu, z, 2);
+        z += __shfl_xor_sync(0xffffffffu, z, 1);
+        if (i < d && l8 == 0) {
+            ws[i] = general_decay(z + p.w0[(size_t)h * d + i], p.decay_rate);
+            bs[i] = sigmoidf(row[4 * (size_t)n + i] + p.a_bias[(size_t)h * d + i]) * ks[i] * inv2;
+        }
+    }
+    __syncthreads();
+    const bool fresh = pos_of(p.ps) == 0;
+    const int c = threadIdx.x % p.cw, rg = threadIdx.x / p.cw, groups = blockDim.x / p.cw;
+    const int per = (d + groups - 1) / groups, i0 = min(d, rg * per), i1 = min(d, i0 + per);
+    float* S = p.state + (size_t)h * d * d;
+    for (int c0 = 0; c0 < d; c0 += p.cw) {
+        const int j = c0 + c;
+        float held = 0.0f;
+        if (j < d && !fresh) {
+#pragma unroll 8
+            for (int i = i0; i < i1; i++) held = fmaf(S[(size_t)i * d + j], ks[i], held);
+        }
+        part[threadIdx.x] = held;
+        __syncthreads();
+        held = 0.0f;
+        for (int g = 0; g < groups; g++) held += part[g * p.cw + c];
+        __syncthreads();
+        float o = 0.0f;
+        if (j < d) {
+            const float v = row[2 * (size_t)n + j];
+            for (int ib = i0; ib < i1; ib += 4) {   // four rows' loads ahead of their stores
+                float old[4], r[4];
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    old[e] = ib + e < i1 && !fresh ? S[(size_t)(ib + e) * d + j] : 0.0f;
+                    r[e] = ib + e < i1 ? row[ib + e] : 0.0f;
+                }
+#pragma unroll
+                for (int e = 0; e < 4; e++)
+                    if (ib + e < i1) {
+                        const float nw = fmaf(-bs[ib + e], held, fmaf(ws[ib + e], old[e], ks[ib + e] * v));
+                        S[(size_t)(ib + e) * d + j] = nw;
+                        o = fmaf(nw, r[e], o);
+                    }
+            }
+        }
+        part[threadIdx.x] = o;
+        __syncthreads();
+        if (rg == 0 && j < d) {
+            o = 0.0f;
+            for (int g = 0; g < groups; g++) o += part[g * p.cw + c];
+            os[j] = o;
+        }
+        __syncthreads();
+    }
+    ss = 0.0f;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) ss += os[j] * os[j];
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)d + p.eps);
+    for (int j = threadIdx.x; j < d; j += blockDim.x)
+        from_f(p.out[(size_t)h * d + j], os[j] * inv * p.w[(size_t)h * d + j] * sigmoidf(row[3 * (size_t)n + j]));
+}
+
 // o / sqrt(mean(o^2) + eps) * w[c] * sigmoid(gate logit) per (token, head): one warp each
 // gate_silu: the gate is silu(logit) instead.  g_ld / out_ld (with H): the gate logits / the output of a token are H * dv
 // columns of a wider row with this pitch; has_out_scale: the output times out_scale
@@ -503,6 +684,7 @@ template <typename AT> struct GatedHeadNormParams {
     int rows, dv;
     int gate_silu, H, g_ld, out_ld, has_out_scale;
     float out_scale;
+    int w_ld;                            // with H: head hh's weights start at w + hh * w_ld (0: one vector for all heads)
 };
 template <typename AT> __global__ void __launch_bounds__(128) gated_headnorm_kernel(const GatedHeadNormParams<AT> p) {
     pdl_launch();
@@ -514,13 +696,14 @@ template <typename AT> __global__ void __launch_bounds__(128) gated_headnorm_ker
     const int t = p.H > 0 ? r / p.H : 0, hh = p.H > 0 ? r % p.H : 0;
     const float* gr = p.g_ld > 0 ? p.graw + (size_t)t * p.g_ld + (size_t)hh * p.dv : p.graw + (size_t)r * p.dv;
     AT* dst = p.out_ld > 0 ? p.out + (size_t)t * p.out_ld + (size_t)hh * p.dv : p.out + (size_t)r * p.dv;
+    const float* w = p.w + (size_t)hh * p.w_ld;
     float ss = 0.0f;
     for (int c = lane; c < p.dv; c += 32) ss += o[c] * o[c];
     ss = warp_sum(ss);
     const float inv = (p.has_out_scale ? p.out_scale : 1.0f) / sqrtf(ss / (float)p.dv + p.eps);
     for (int c = lane; c < p.dv; c += 32) {
         const float sg = 1.0f / (1.0f + expf(-gr[c]));
-        from_f(dst[c], o[c] * inv * p.w[c] * (p.gate_silu ? gr[c] * sg : sg));
+        from_f(dst[c], o[c] * inv * w[c] * (p.gate_silu ? gr[c] * sg : sg));
     }
 }
 

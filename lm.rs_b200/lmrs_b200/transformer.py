@@ -24,6 +24,7 @@ class ModelType(IntEnum):  # src/transformer.rs:50-55
     TUDATAR = 4   # a folder model: delta-rule / latent-attention / windowed-attention layers with routed experts
     RUPENEX = 5   # a folder model: state-space / sink-attention layers, dense or routed feed-forward, layer-normed sublayer outputs
     BADEPEL = 6   # a folder model: several residual streams; windowed attention beside gated linear attention, delta-rule layers, dense or routed feed-forward
+    BOLAPEL = 7   # a folder model: generalized-delta-rule / chunked sigmoid-attention layers with token shift, norms around every sublayer
 
 
 class QuantType(IntEnum):  # src/quantization.rs:1-6
