@@ -17,7 +17,7 @@
 //                             decay per head instead of per key channel; or without the correction (gated linear attention:
 //                             S <- diag(g) S + k v^T); or with a decay and a removal rate per key channel (generalized delta
 //                             rule: S <- diag(w) S - (a u)(u^T S) + k v^T, u the unit key, both terms from the old S)
-//   general_delta_pre_kernel  what that last form needs per token and key channel: decays, removal vectors, the query's product
+//   general_delta_pre_kernel  what that last form needs per token and key channel: losses (1 - decay), removal vectors, the query's product
 //                             with the removal vector
 //   general_delta_step_kernel one token of it, from the projected row to the gated output row: decays, update, read-out, norm, gate
 //   gated_headnorm_kernel     o / rms(o) * w * sigmoid(gate) per head, in the operand type
@@ -344,7 +344,7 @@ static __global__ void __launch_bounds__(256) delta_decay_kernel(const DeltaDeca
 constexpr int DELTA_TB = 8, DELTA_THREADS = 128, DELTA_MAX_DK = 512;
 struct DeltaScanParams {
     const float* qkv; int ld;   // [T][C]: q at 0, k at G*dk, v at 2*G*dk
-    const float* decay;         // [T][H*dk]
+    const float* decay;         // [T][H*dk] (SCAN_DELTA_HEAD: [T][H]; SCAN_GENERAL: losses)
     const float* beta;          // [T][H]
     float* state;               // [H][dk][dv]
     float* out;                 // [T][H*dv]
@@ -357,8 +357,10 @@ struct DeltaScanParams {
 // one decay per head (decay is [T][H]).  SCAN_PLAIN: no correction and no write strength, S <- diag(g) S + k v^T, o = S^T q
 // (gated linear attention): one pass over the registers and one lane reduction per token.  SCAN_GENERAL: with a removal vector
 // b per token (rem; general_delta_pre_kernel folds the unit key's length into it) and s = S^T k from the OLD state,
-// S <- diag(g) S + k v^T - b s^T.  Nothing but that last subtraction waits for s: M = diag(g) S + k v^T and M^T q are formed
-// while s is being reduced, and o = M^T q - (q . b) s with the scalar q . b given in beta -- one round of lane reductions per token.
+// S <- diag(1 - l) S + k v^T - b s^T, where decay holds the losses l = 1 - g instead of the decays g (a decay a hair below one
+// keeps its relative precision that way, and the state loses no more than the rounding of one addition per token).  Nothing but
+// the last subtraction waits for s: M = S + (k v^T - diag(l) S) and M^T q are formed while s is being reduced, and
+// o = M^T q - (q . b) s with the scalar q . b given in beta -- one round of lane reductions per token.
 enum { SCAN_DELTA = 0, SCAN_DELTA_HEAD = 1, SCAN_PLAIN = 2, SCAN_GENERAL = 3 };
 // (rows per lane NR, lanes per column LPC) for a key size: NR * LPC >= dk.  A warp issues dependent instructions only every few
 // cycles, so the split favours many lanes per column (more warps per scheduler, shorter chains) over few
@@ -461,8 +463,8 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
                     const float4 q4 = *reinterpret_cast<const float4*>(qs + tt * dkp + i);
                     r0 = fmaf(S[4 * r4], k4.x, r0); r1 = fmaf(S[4 * r4 + 1], k4.y, r1);
                     r2 = fmaf(S[4 * r4 + 2], k4.z, r2); r3 = fmaf(S[4 * r4 + 3], k4.w, r3);
-                    S[4 * r4] = fmaf(S[4 * r4], g4.x, k4.x * v); S[4 * r4 + 1] = fmaf(S[4 * r4 + 1], g4.y, k4.y * v);
-                    S[4 * r4 + 2] = fmaf(S[4 * r4 + 2], g4.z, k4.z * v); S[4 * r4 + 3] = fmaf(S[4 * r4 + 3], g4.w, k4.w * v);
+                    S[4 * r4] += fmaf(-S[4 * r4], g4.x, k4.x * v); S[4 * r4 + 1] += fmaf(-S[4 * r4 + 1], g4.y, k4.y * v);
+                    S[4 * r4 + 2] += fmaf(-S[4 * r4 + 2], g4.z, k4.z * v); S[4 * r4 + 3] += fmaf(-S[4 * r4 + 3], g4.w, k4.w * v);
                     o0 = fmaf(S[4 * r4], q4.x, o0); o1 = fmaf(S[4 * r4 + 1], q4.y, o1);
                     o2 = fmaf(S[4 * r4 + 2], q4.z, o2); o3 = fmaf(S[4 * r4 + 3], q4.w, o3);
                 }
@@ -539,15 +541,15 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
 // ---- generalized delta rule ---------------------------------------------------------------------------------------------------
 // The projected row is [r (H*d) | k (H*d) | v (H*d) | gate logits (H*d) | removal logits (H*d) | decay latent]; z holds the decay
 // logits (second half of the low-rank projection, bias added).  Per token, head and key channel
-//     decay = exp(-decay_rate * sigmoid(z))          removal rate a = sigmoid(removal logit + bias)
+//     decay = exp(-decay_rate * sigmoid(z)), kept as the loss 1 - decay          removal rate a = sigmoid(removal logit + bias)
 // and with u = k / sqrt(sum k^2 + 1e-6) the state update S <- diag(decay) S - (a u)(u^T S) + k v^T is what delta_scan_kernel's
 // SCAN_GENERAL does with b = a k / (sum k^2 + 1e-6) as the removal vector and s = S^T k.  Also the scalar r . b.  One warp per
-// (token, head); decays replace the logits in place.
+// (token, head); losses replace the logits in place.
 DN_DEVINL float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
-DN_DEVINL float general_decay(float z, float rate) { return expf(-rate * sigmoidf(z)); }
+DN_DEVINL float general_loss(float z, float rate) { return -expm1f(-rate * sigmoidf(z)); }
 struct GeneralDeltaPreParams {
     const float* proj; int ld;
-    float* z;                  // [T][H*d] decay logits in, decays out
+    float* z;                  // [T][H*d] decay logits in, losses out
     const float* a_bias;       // [H*d]
     float* rem; float* rb;     // [T][H*d], [T][H]
     int T, H, d;
@@ -569,7 +571,7 @@ static __global__ void __launch_bounds__(128) general_delta_pre_kernel(const Gen
         const float b = sigmoidf(row[4 * n + i] + p.a_bias[(size_t)h * p.d + i]) * row[n + i] * inv2;
         rb = fmaf(row[i], b, rb);
         p.rem[o + i] = b;
-        p.z[o + i] = general_decay(p.z[o + i], p.decay_rate);
+        p.z[o + i] = general_loss(p.z[o + i], p.decay_rate);
     }
     rb = warp_sum(rb);
     if (lane == 0) p.rb[(size_t)t * p.H + h] = rb;
@@ -597,7 +599,7 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
     const int h = blockIdx.x, d = p.d, n = p.H * d;
     float* lat = gd_sm;            // [ra]
     float* ks = lat + p.ra;        // [d] key
-    float* ws = ks + d;            // [d] decays
+    float* ws = ks + d;            // [d] losses
     float* bs = ws + d;            // [d] removal vector
     float* os = bs + d;            // [d] read-out
     float* part = os + d;          // [blockDim.x] sums of the row groups
@@ -618,7 +620,7 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
         z += __shfl_xor_sync(0xffffffffu, z, 2);
         z += __shfl_xor_sync(0xffffffffu, z, 1);
         if (i < d && l8 == 0) {
-            ws[i] = general_decay(z + p.w0[(size_t)h * d + i], p.decay_rate);
+            ws[i] = general_loss(z + p.w0[(size_t)h * d + i], p.decay_rate);
             bs[i] = sigmoidf(row[4 * (size_t)n + i] + p.a_bias[(size_t)h * d + i]) * ks[i] * inv2;
         }
     }
@@ -652,7 +654,7 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
 #pragma unroll
                 for (int e = 0; e < 4; e++)
                     if (ib + e < i1) {
-                        const float nw = fmaf(-bs[ib + e], held, fmaf(ws[ib + e], old[e], ks[ib + e] * v));
+                        const float nw = fmaf(-bs[ib + e], held, old[e] + fmaf(-ws[ib + e], old[e], ks[ib + e] * v));
                         S[(size_t)(ib + e) * d + j] = nw;
                         o = fmaf(nw, r[e], o);
                     }
