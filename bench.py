@@ -147,6 +147,9 @@ def bench_arch(args):
     --arch badepel: that architecture (delta-rule layers and windowed attention beside gated linear attention, several residual
     streams, dense and routed feed-forwards in turn) and Tudatar, the closest folder model (a delta-rule mixer, windowed
     attention with whole-row q/k norms, routed experts), at the same layer shape.
+    --arch bolapel: that architecture (three generalized-delta-rule layers for every chunked sigmoid-attention layer, dense
+    feed-forwards) and Tudatar, the closest folder model (a delta rule with a decay per key channel, windowed attention, norms on
+    both sides of every sublayer; its chosen experts are as wide as the dense feed-forward), at the same layer shape.
     Prefill: device time (CUDA events on the handle's stream) of one pass over T prompt tokens.  Decode: device time of K
     HBM-resident steps at positions P.. after a P-token prompt, and the same loop end to end through forward_argmax.  Every
     step streams the whole weight set (larger than L2), so no flush is needed between steps."""
@@ -272,7 +275,20 @@ def bench_arch(args):
         folder_model("badepel", bcfg, md.write_random_badepel, md.badepel_matmul_flops_per_token(bcfg) - head_flops,
                      lambda T: md.badepel_mixer_flops(bcfg, T), md.badepel_param_bytes(bcfg), kvb,
                      "bf16 weights and operands, f32 accumulation; f32 residual streams, caches, recurrent states, norms, router")
-    if args.arch in ("tudatar", "rupenex", "badepel"):
+    if args.arch == "bolapel":
+        ocfg = md.bolapel_config(a.dim, a.n_layers, a.vocab_size, heads=a.n_heads, kv_heads=a.n_kv_heads, head_dim=a.head_size, chunk=1024,
+                                 delta_dim=args.arch_delta_dim, rank=64, ff=a.hidden_dim)
+        kvb = 0
+        for L in ocfg["layers"]:
+            mx = L["mixer"]
+            if L["type"] == "general_delta":
+                kvb += 2 * mx["heads"] * mx["dim"] * mx["dim"] * 4   # the state is read and written
+            else:
+                kvb += 2 * ((P + K // 2) % mx["mask"]["size"]) * mx["kv_heads"] * mx["dim"] * 4
+        folder_model("bolapel", ocfg, md.write_random_bolapel, md.bolapel_matmul_flops_per_token(ocfg) - head_flops,
+                     lambda T: md.bolapel_mixer_flops(ocfg, T), md.bolapel_param_bytes(ocfg), kvb,
+                     "bf16 weights and operands, f32 accumulation; f32 residual, caches, recurrent states, norms")
+    if args.arch in ("tudatar", "rupenex", "badepel", "bolapel"):
         top = 4
         tcfg = md.tudatar_config(a.dim, a.n_layers, a.vocab_size, heads=a.n_heads, kv_heads=a.n_kv_heads, head_dim=a.head_size,
                                  delta_heads=max(1, a.dim // 128), delta_dim=128, experts=args.arch_experts, top=top,
@@ -289,6 +305,25 @@ def bench_arch(args):
         folder_model("tudatar", tcfg, md.write_random_tudatar, md.tudatar_matmul_flops_per_token(tcfg) - head_flops,
                      lambda T: md.tudatar_mixer_flops(tcfg, T), md.tudatar_param_bytes(tcfg), kvb,
                      "bf16 weights and operands, f32 accumulation; f32 caches, recurrent state, norms, router")
+    if args.arch == "bolapel":
+        clocks = sampler.stop()
+        g = out["bolapel"]["decode"]
+        dd = args.arch_delta_dim
+        print(json.dumps({
+            "metric": f"decode tok/s Bolapel bf16 at the layer shape of {args.model} (prefill and Tudatar of the same shape in 'arch')",
+            "value": g["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": Wm, "ms_per_step": g["ms_per_step"],
+            "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"model": f"Bolapel {a.n_layers} layers (3 x generalized delta rule, chunked sigmoid attention, ...; every second attention layer on the "
+                                f"keys and values of the one before), dense ff {a.hidden_dim}, width {a.dim}, {a.n_heads}/{a.n_kv_heads} heads of "
+                                f"{a.head_size}, chunk 1024, delta rule {a.dim // dd} heads of {dd} x {dd}, vocab {a.vocab_size}",
+                       "first_pos": P, "batch": 1, "prefill_lengths": lens,
+                       "l2": "inputs larger than L2 (the weight set is streamed every step); no flush needed"},
+            "e2e": {"value": g["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 16, "d2h_bytes_per_step": 4,
+                    "api": "forward_argmax(token, pos) -> next token"},
+            "gpu_launches": launches_total[0], "clocks": clocks,
+            "peaks": {"hbm_gb_s": peak_hbm, "hbm_source": peak_src, "bf16_tflops": peak_tf, "bf16_source": tf_src},
+            "arch": out}))
+        return
     if args.arch == "badepel":
         clocks = sampler.stop()
         g = out["badepel"]["decode"]
@@ -399,9 +434,10 @@ def main():
     ap.add_argument("--pos", type=int, default=512, help="prompt length / first decode position")
     ap.add_argument("--cpu-steps", type=int, default=16, help="decode steps of the bounded cpu_baseline sample")
     ap.add_argument("--parity-steps", type=int, default=4, help="greedy decode steps replayed on the CPU oracle (0: skip the parity block)")
-    ap.add_argument("--arch-experts", type=int, default=16, help="--arch tudatar / rupenex / badepel: experts per layer (4 are chosen)")
+    ap.add_argument("--arch-experts", type=int, default=16, help="--arch tudatar / rupenex / badepel / bolapel (its Tudatar): experts per layer (4 are chosen)")
     ap.add_argument("--arch-streams", type=int, default=4, help="--arch badepel: residual streams per token")
-    ap.add_argument("--arch", default="", choices=["", "genetar", "tudatar", "rupenex", "badepel"],
+    ap.add_argument("--arch-delta-dim", type=int, default=64, help="--arch bolapel: key and value size of a delta-rule head")
+    ap.add_argument("--arch", default="", choices=["", "genetar", "tudatar", "rupenex", "badepel", "bolapel"],
                     help="instead of the default workload: prefill and decode throughput of this folder-model architecture (random "
                          "bf16 weights at the layer shape of --model) beside the LMRS Q8_0 Llama of the same shape")
     ap.add_argument("--arch-layers", type=int, default=0, help="--arch: number of layers (0: as many as --model has)")

@@ -1,6 +1,6 @@
 """Model folders (config.json + model.safetensors) for the architectures the library opens by name: a writer, the
-tensor tables of the Genetar, Tudatar, Rupenex and Badepel architectures, and random bf16 weights of a given shape for benchmarks and
-smoke runs.
+tensor tables of the Genetar, Tudatar, Rupenex, Badepel and Bolapel architectures, and random bf16 weights of a given shape for
+benchmarks and smoke runs.
 
 safetensors layout: 8-byte little-endian header length, that many bytes of JSON (name -> dtype, shape, data_offsets
 relative to the end of the header), then the tensor data.
@@ -458,4 +458,90 @@ def write_random_badepel(folder, cfg, seed=0):
     write_random(folder, cfg, badepel_tensors(cfg), seed)
     with open(os.path.join(folder, "config.json"), "w") as f:
         json.dump(written_badepel_config(cfg), f)
+    return folder
+
+
+# ---- Bolapel ---------------------------------------------------------------------------------------------------------------
+def bolapel_config(width, n_layers, vocab, *, heads=16, kv_heads=4, head_dim=64, vdim=None, chunk=1024, rot_dims=None, delta_heads=None, delta_dim=64,
+                   rank=64, ff=8192, softcap=30.0, eps=1e-5, pattern=("general_delta", "general_delta", "general_delta", "attention"), share_kv=True):
+    """layers cycle through `pattern`; with share_kv every second attention layer reads the keys and values of the attention
+    layer before it; the inner size of the delta rule is the model width unless delta_heads says otherwise"""
+    layers, lender = [], None
+    for i in range(n_layers):
+        kind = pattern[i % len(pattern)]
+        if kind == "general_delta":
+            m = {"heads": delta_heads or width // delta_dim, "dim": delta_dim, "rank": rank}
+        else:
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": vdim or head_dim, "scale": 1.0 / math.sqrt(head_dim), "mask": {"size": chunk},
+                 "rot": {"base": 10000.0, "dims": rot_dims or head_dim // 2}}
+            if share_kv and lender is not None:
+                m["kv_from"], lender = lender, None
+            else:
+                lender = i
+        layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None})
+    return {"architecture": "Bolapel", "width": width, "vocab": vocab, "norm": {"eps": eps}, "logit_softcap": softcap, "layers": layers}
+
+
+def bolapel_tensors(cfg):
+    """[(name, shape, kind)] -- the rank of the delta rule's decay projection is a tensor shape, not configuration: the writer takes
+    it from the hint `rank` that bolapel_config leaves in the mixer entry"""
+    w = cfg["width"]
+    out = [("embed", (cfg["vocab"], w), "table")]
+    for i, L in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", L["mixer"], L.get("mlp")
+        q = p + "mix."
+        out += [(p + "norm1", (w,), "ones"), (p + "norm1b", (w,), "ones"), (p + "shift", (w,), "small")]
+        if L["type"] == "general_delta":
+            n, r = m["heads"] * m["dim"], m.get("rank", 16)
+            out += [(q + s, (n, w), "matrix") for s in ("r", "k", "v", "g", "a")]
+            out += [(q + "a.b", (n,), "shift"), (q + "w1", (r, w), "matrix"), (q + "w2", (n, r), "matrix"), (q + "w0", (n,), "rate"),
+                    (q + "norm", (n,), "ones"), (q + "o", (w, n), "matrix")]
+        else:
+            H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            out += [(q + "q", (H * dk, w), "matrix"), (q + "q.norm", (dk,), "ones"), (q + "pb", (H,), "rate"), (q + "g", (H, w), "matrix"),
+                    (q + "o", (w, H * dv), "matrix")]
+            if m.get("kv_from") is None:
+                out += [(q + "k", (G * dk, w), "matrix"), (q + "v", (G * dv, w), "matrix"), (q + "k.norm", (dk,), "ones")]
+        if f:
+            out += [(p + "norm2", (w,), "ones"), (p + "norm2b", (w,), "ones"), (p + "mlp.gate", (f["ff"], w), "matrix"),
+                    (p + "mlp.up", (f["ff"], w), "matrix"), (p + "mlp.down", (w, f["ff"]), "matrix")]
+    return out + [("final.norm", (w,), "ones"), ("head", (cfg["vocab"], w), "matrix")]
+
+
+def bolapel_param_bytes(cfg, bytes_per_weight=2):
+    """bytes a decode step streams: every matrix once, one embedding row"""
+    return sum((shape[1] if kind == "table" else int(np.prod(shape))) * bytes_per_weight for _, shape, kind in bolapel_tensors(cfg))
+
+
+def bolapel_matmul_flops_per_token(cfg):
+    return sum(2 * int(np.prod(shape)) for _, shape, kind in bolapel_tensors(cfg) if kind == "matrix")
+
+
+def bolapel_mixer_flops(cfg, T):
+    """FLOPs of the sequence mixers' cores over a prompt of T tokens: attention inside the chunks, the delta-rule scan (what the
+    key holds, decay and write, removal, read-out: 10 per state entry and token)"""
+    total = 0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        if L["type"] == "general_delta":
+            total += 10 * m["heads"] * m["dim"] * m["dim"] * T
+        else:
+            c = (m.get("mask") or {}).get("size", 0) or T
+            pairs = (T // c) * (c * (c + 1) // 2) + (T % c) * (T % c + 1) // 2
+            total += 2 * m["heads"] * (m["dim"] + m["vdim"]) * pairs
+    return total
+
+
+def written_bolapel_config(cfg):
+    """config.json without the writer's hints"""
+    c = json.loads(json.dumps(cfg))
+    for L in c["layers"]:
+        L["mixer"].pop("rank", None)
+    return c
+
+
+def write_random_bolapel(folder, cfg, seed=0):
+    write_random(folder, cfg, bolapel_tensors(cfg), seed)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(written_bolapel_config(cfg), f)
     return folder
