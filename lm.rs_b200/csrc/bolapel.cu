@@ -60,7 +60,7 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
     unsigned int* counter = nullptr;
     uint32_t next_pos = 0;         // where the recurrent states and shift rows stand
     // scratch for `cap` rows
-    float *proj = nullptr, *qa = nullptr, *gate = nullptr, *z = nullptr, *rem = nullptr, *rb = nullptr, *fo = nullptr, *yf = nullptr, *part = nullptr, *inv = nullptr;
+    float *proj = nullptr, *qa = nullptr, *gate = nullptr, *z = nullptr, *rec = nullptr, *fo = nullptr, *yf = nullptr, *part = nullptr, *inv = nullptr;
     AT *h = nullptr, *lat = nullptr, *att = nullptr, *act = nullptr;
     int max_proj = 0, max_ra = 0, max_q = 0, max_n = 0, max_H = 0, max_dv = 0, max_att = 0, max_ff = 0;
     // test / measurement overrides: lanes per state column of the scan, one-token steps through the many-token kernels
@@ -206,16 +206,22 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         if (rows <= cap) return 0;
         drop_graphs();   // captured launches point into the old scratch
         for (void* p : {(void*)x, (void*)hn, (void*)d_rows, (void*)h, (void*)lat, (void*)att, (void*)act, (void*)proj, (void*)qa, (void*)gate, (void*)z,
-                        (void*)rem, (void*)rb, (void*)fo, (void*)yf, (void*)part, (void*)inv})
+                        (void*)rec, (void*)fo, (void*)yf, (void*)part, (void*)inv})
             dfree(p);
         x = nullptr; hn = nullptr; d_rows = nullptr; h = nullptr; lat = nullptr; att = nullptr; act = nullptr; proj = nullptr; qa = nullptr; gate = nullptr;
-        z = nullptr; rem = nullptr; rb = nullptr; fo = nullptr; yf = nullptr; part = nullptr; inv = nullptr;
+        z = nullptr; rec = nullptr; fo = nullptr; yf = nullptr; part = nullptr; inv = nullptr;
         cap = 0;
         int max_heads = 1;
-        for (const Layer& L : layers) max_heads = std::max(max_heads, L.c.H);
+        size_t max_rec = 0;   // floats of a four-token block's records
+        for (const Layer& L : layers) {
+            max_heads = std::max(max_heads, L.c.H);
+            int nr, lpc;
+            scan_shape(L.c.d, &nr, &lpc);
+            if (L.c.kind == BO_DELTA) max_rec = std::max(max_rec, (size_t)L.c.H * gd_record(nr * lpc));
+        }
         if (dalloc(&x, rows * width) || dalloc(&hn, rows * width) || dalloc(&d_rows, rows) || dalloc(&h, rows * width) || dalloc(&lat, rows * max_ra) ||
             dalloc(&att, rows * max_att) || dalloc(&act, rows * max_ff) || dalloc(&proj, rows * max_proj) || dalloc(&qa, rows * max_q) ||
-            dalloc(&gate, rows * max_heads) || dalloc(&z, rows * max_n) || dalloc(&rem, rows * max_n) || dalloc(&rb, rows * max_heads) ||
+            dalloc(&gate, rows * max_heads) || dalloc(&z, rows * max_n) || dalloc(&rec, (rows + GD_BLOCK - 1) / GD_BLOCK * max_rec) ||
             dalloc(&fo, rows * max_n) || dalloc(&yf, rows * width) || dalloc(&part, (size_t)std::max(max_H, 1) * MAX_SPLIT * (max_dv + 2)) || dalloc(&inv, rows))
             return 1;
         cap = rows;
@@ -274,25 +280,34 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         EpiParams<AT> e{}; e.out = proj; e.ldo = L.in_rows; e.scale = 1.0f;
         return this->template matmul<EPI_STORE>(st, T, h, width, L.w_in, nullptr, width, L.in_rows, e);
     }
-    template <int NR, int LPC> int launch_scan(cudaStream_t st, const DeltaScanParams& sp) {
-        constexpr int cols = DELTA_THREADS / LPC;
-        const size_t smem = delta_scan_smem(NR, LPC, SCAN_GENERAL);
-        if (optin(delta_scan_kernel<NR, LPC, SCAN_GENERAL>, smem)) return 1;
-        return launch_k("delta_scan_kernel", st, pdl_now, delta_scan_kernel<NR, LPC, SCAN_GENERAL>, dim3((sp.dv + cols - 1) / cols, sp.H), dim3(DELTA_THREADS), smem, sp);
+    // rows per lane and lanes per column of the scan for a key size
+    void scan_shape(int d, int* nr, int* lpc) const {
+        if (d <= 32) { *nr = 4; *lpc = 8; }
+        else if (d <= 64) { *nr = 8; *lpc = 8; if (scan_lanes == 16) { *nr = 4; *lpc = 16; } }
+        else if (d <= 128) { *nr = 8; *lpc = 16; if (scan_lanes == 32) { *nr = 4; *lpc = 32; } }
+        else if (d <= 256) { *nr = 8; *lpc = 32; }
+        else { *nr = 16; *lpc = 32; }
     }
-    int scan(cudaStream_t st, const DeltaScanParams& sp) {
-        int nr, lpc;
-        delta_scan_shape(sp.dk, &nr, &lpc);
-        if (sp.dk > 32 && sp.dk <= 64) {
-            if (scan_lanes == 4) return launch_scan<16, 4>(st, sp);
-            if (scan_lanes == 16) return launch_scan<4, 16>(st, sp);
-        }
-        if (nr == 16 && lpc == 1) return launch_scan<16, 1>(st, sp);
-        if (nr == 16 && lpc == 2) return launch_scan<16, 2>(st, sp);
+    template <int NR, int LPC> int launch_scan(cudaStream_t st, const GeneralDeltaScanParams& sp) {
+        constexpr int cols = GD_THREADS / LPC;
+        const size_t smem = general_delta_scan_smem<NR, LPC>();
+        if (optin(general_delta_scan_kernel<NR, LPC>, smem)) return 1;
+        return launch_k("general_delta_scan_kernel", st, pdl_now, general_delta_scan_kernel<NR, LPC>, dim3((sp.d + cols - 1) / cols, sp.H), dim3(GD_THREADS), smem, sp);
+    }
+    int scan(cudaStream_t st, int nr, int lpc, const GeneralDeltaScanParams& sp) {
+        if (nr == 4 && lpc == 8) return launch_scan<4, 8>(st, sp);
         if (nr == 8 && lpc == 8) return launch_scan<8, 8>(st, sp);
+        if (nr == 4 && lpc == 16) return launch_scan<4, 16>(st, sp);
         if (nr == 8 && lpc == 16) return launch_scan<8, 16>(st, sp);
+        if (nr == 4 && lpc == 32) return launch_scan<4, 32>(st, sp);
         if (nr == 8 && lpc == 32) return launch_scan<8, 32>(st, sp);
         return launch_scan<16, 32>(st, sp);
+    }
+
+    template <int RPT> int launch_step(cudaStream_t st, const GeneralDeltaStepParams<AT, WT>& p, int threads) {
+        const size_t smem = ((size_t)p.ra + 5 * p.d + threads) * 4;
+        if (optin(general_delta_step_kernel<AT, WT, RPT>, smem)) return 1;
+        return launch_k("general_delta_step_kernel", st, pdl_now, general_delta_step_kernel<AT, WT, RPT>, dim3(p.H), dim3(threads), smem, p);
     }
 
     // leaves the row that the output projection multiplies in att
@@ -307,22 +322,24 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
             p.cw = 32;
             while (p.cw < c.d) p.cw *= 2;
             const int threads = p.cw * std::min(1024 / p.cw, (c.d + 3) / 4);   // about four state rows per thread
-            const size_t smem = ((size_t)c.ra + 4 * c.d + threads) * 4;
-            if (optin(general_delta_step_kernel<AT, WT>, smem)) return 1;
-            return launch_k("general_delta_step_kernel", st, pdl_now, general_delta_step_kernel<AT, WT>, dim3(c.H), dim3(threads), smem, p);
+            const int per = (c.d + threads / p.cw - 1) / (threads / p.cw);
+            if (per <= 4) return launch_step<4>(st, p, threads);
+            if (per <= 16) return launch_step<16>(st, p, threads);
+            return launch_step<0>(st, p, threads);
         }
         CastColsParams<AT> cp{};   // the low-rank decay latent in the operand type, for the second half of that projection
         cp.in = proj + 5 * (size_t)n; cp.ld = L.in_rows; cp.out = lat; cp.ldo = c.ra; cp.n = c.ra; cp.total = T * c.ra; cp.tanh_first = 1;
         if (launch_k("cast_cols_kernel", st, pdl_now, cast_cols_kernel<AT>, dim3((cp.total + 255) / 256), dim3(256), 0, cp)) return 1;
         EpiParams<AT> ez{}; ez.out = z; ez.ldo = n; ez.scale = 1.0f; ez.bias = L.w0;
         if (this->template matmul<EPI_STORE>(st, T, lat, c.ra, L.w2, nullptr, c.ra, n, ez)) return 1;
+        int nr, lpc;
+        scan_shape(c.d, &nr, &lpc);
         GeneralDeltaPreParams pp{};
-        pp.proj = proj; pp.ld = L.in_rows; pp.z = z; pp.a_bias = L.a_bias; pp.rem = rem; pp.rb = rb; pp.T = T; pp.H = c.H; pp.d = c.d; pp.decay_rate = decay_rate;
-        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3((T * c.H + 3) / 4), dim3(128), 0, pp)) return 1;
-        DeltaScanParams sp{};
-        sp.qkv = proj; sp.ld = L.in_rows; sp.decay = z; sp.rem = rem; sp.beta = rb; sp.state = L.state; sp.out = fo;
-        sp.T = T; sp.H = c.H; sp.G = c.H; sp.dk = c.d; sp.dv = c.d; sp.ps = ps;
-        if (scan(st, sp)) return 1;
+        pp.proj = proj; pp.ld = L.in_rows; pp.z = z; pp.a_bias = L.a_bias; pp.rec = rec; pp.T = T; pp.H = c.H; pp.d = c.d; pp.dp = nr * lpc; pp.decay_rate = decay_rate;
+        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3(((T + GD_BLOCK - 1) / GD_BLOCK * c.H + 3) / 4), dim3(128), 0, pp)) return 1;
+        GeneralDeltaScanParams sp{};
+        sp.rec = rec; sp.v = proj + 2 * (size_t)n; sp.ld = L.in_rows; sp.state = L.state; sp.out = fo; sp.T = T; sp.H = c.H; sp.d = c.d; sp.ps = ps;
+        if (scan(st, nr, lpc, sp)) return 1;
         GatedHeadNormParams<AT> gp{};
         gp.o = fo; gp.graw = proj + 3 * (size_t)n; gp.w = L.onorm; gp.w_ld = c.d; gp.eps = info.eps; gp.out = att; gp.rows = T * c.H; gp.dv = c.d; gp.H = c.H;
         gp.g_ld = L.in_rows;

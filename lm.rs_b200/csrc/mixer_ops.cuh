@@ -15,10 +15,10 @@
 //   delta_scan_kernel         S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q, token after token, the
 //                             state matrix of a head spread over the registers of the threads that own its columns; with one
 //                             decay per head instead of per key channel; or without the correction (gated linear attention:
-//                             S <- diag(g) S + k v^T); or with a decay and a removal rate per key channel (generalized delta
-//                             rule: S <- diag(w) S - (a u)(u^T S) + k v^T, u the unit key, both terms from the old S)
-//   general_delta_pre_kernel  what that last form needs per token and key channel: losses (1 - decay), removal vectors, the query's product
-//                             with the removal vector
+//                             S <- diag(g) S + k v^T)
+//   general_delta_pre_kernel  generalized delta rule S <- diag(w) S - (a u)(u^T S) + k v^T (u the unit key, both terms from the old
+//                             S): what the scan below needs per block of four tokens
+//   general_delta_scan_kernel the rule, four tokens at a time: one round of lane reductions per block
 //   general_delta_step_kernel one token of it, from the projected row to the gated output row: decays, update, read-out, norm, gate
 //   gated_headnorm_kernel     o / rms(o) * w * sigmoid(gate) per head, in the operand type
 //   ssm_pre_kernel            state-space recurrence with one decay per head: short causal convolution + bias + SiLU over the
@@ -344,24 +344,18 @@ static __global__ void __launch_bounds__(256) delta_decay_kernel(const DeltaDeca
 constexpr int DELTA_TB = 8, DELTA_THREADS = 128, DELTA_MAX_DK = 512;
 struct DeltaScanParams {
     const float* qkv; int ld;   // [T][C]: q at 0, k at G*dk, v at 2*G*dk
-    const float* decay;         // [T][H*dk] (SCAN_DELTA_HEAD: [T][H]; SCAN_GENERAL: losses)
+    const float* decay;         // [T][H*dk]
     const float* beta;          // [T][H]
     float* state;               // [H][dk][dv]
     float* out;                 // [T][H*dv]
     int T, H, G, dk, dv;
     PosSrc ps;
     float q_scale;              // the read-out times this constant (0: none)
-    const float* rem;           // SCAN_GENERAL: [T][H*dk] removal vectors
 };
 // what the scan computes per token.  SCAN_DELTA: the rule above with a decay per key channel.  SCAN_DELTA_HEAD: the same with
 // one decay per head (decay is [T][H]).  SCAN_PLAIN: no correction and no write strength, S <- diag(g) S + k v^T, o = S^T q
-// (gated linear attention): one pass over the registers and one lane reduction per token.  SCAN_GENERAL: with a removal vector
-// b per token (rem; general_delta_pre_kernel folds the unit key's length into it) and s = S^T k from the OLD state,
-// S <- diag(1 - l) S + k v^T - b s^T, where decay holds the losses l = 1 - g instead of the decays g (a decay a hair below one
-// keeps its relative precision that way, and the state loses no more than the rounding of one addition per token).  Nothing but
-// the last subtraction waits for s: M = S + (k v^T - diag(l) S) and M^T q are formed while s is being reduced, and
-// o = M^T q - (q . b) s with the scalar q . b given in beta -- one round of lane reductions per token.
-enum { SCAN_DELTA = 0, SCAN_DELTA_HEAD = 1, SCAN_PLAIN = 2, SCAN_GENERAL = 3 };
+// (gated linear attention): one pass over the registers and one lane reduction per token.
+enum { SCAN_DELTA = 0, SCAN_DELTA_HEAD = 1, SCAN_PLAIN = 2 };
 // (rows per lane NR, lanes per column LPC) for a key size: NR * LPC >= dk.  A warp issues dependent instructions only every few
 // cycles, so the split favours many lanes per column (more warps per scheduler, shorter chains) over few
 inline void delta_scan_shape(int dk, int* nr, int* lpc) {
@@ -372,7 +366,7 @@ inline void delta_scan_shape(int dk, int* nr, int* lpc) {
     else if (dk <= 256) { *nr = 8; *lpc = 32; }
     else { *nr = 16; *lpc = 32; }
 }
-inline size_t delta_scan_smem(int nr, int lpc, int mode = SCAN_DELTA) { return (size_t)2 * DELTA_TB * ((mode == SCAN_GENERAL ? 4 : 3) * nr * lpc + DELTA_THREADS / lpc + 4) * 4; }
+inline size_t delta_scan_smem(int nr, int lpc) { return (size_t)2 * DELTA_TB * (3 * nr * lpc + DELTA_THREADS / lpc + 4) * 4; }
 DN_DEVINL void cp_async4_zfill(void* smem_dst, const void* gsrc, bool valid) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(smem_dst);
     const int n = valid ? 4 : 0;
@@ -383,8 +377,7 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
     pdl_launch();
     pdl_wait();
     constexpr int cols = DELTA_THREADS / LPC, dkp = NR * LPC;   // dkp: rows the lanes cover (>= dk, a multiple of 4)
-    constexpr int NA = MODE == SCAN_GENERAL ? 4 : 3;            // staged vectors of dkp entries per token: q, k, decays [, removal]
-    constexpr int blk = DELTA_TB * (NA * dkp + cols + 4);       // floats per staging buffer
+    constexpr int blk = DELTA_TB * (3 * dkp + cols + 4);                   // floats per staging buffer
     const int h = blockIdx.y, g = h / (p.H / p.G);
     const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC, j = blockIdx.x * cols + jl;
     const bool col_ok = j < p.dv;
@@ -392,12 +385,12 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
     const int vq = 2 * p.G * p.dk;
     // 16-byte copies when every row piece starts on a 16-byte boundary
     const bool vec = (p.dk & 3) == 0 && (p.ld & 3) == 0 && ((p.H * p.dk) & 3) == 0 && (reinterpret_cast<uintptr_t>(p.qkv) & 15) == 0 &&
-                     (reinterpret_cast<uintptr_t>(p.decay) & 15) == 0 && (MODE != SCAN_GENERAL || (reinterpret_cast<uintptr_t>(p.rem) & 15) == 0);
+                     (reinterpret_cast<uintptr_t>(p.decay) & 15) == 0;
     auto stage = [&](int t0, int buf) {
         float* qs = ds_sm + (size_t)buf * blk;     // [TB][dkp]
         float* ks = qs + DELTA_TB * dkp;
         float* gs = ks + DELTA_TB * dkp;
-        float* vs = qs + NA * DELTA_TB * dkp;      // [TB][cols]
+        float* vs = gs + DELTA_TB * dkp;           // [TB][cols]
         float* bs = vs + DELTA_TB * cols;          // [TB]
         const int nt = min(DELTA_TB, p.T - t0);
         if (vec) {
@@ -409,7 +402,6 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
                 cp_async16_zfill(qs + tt * dkp + i, ok ? row + g * p.dk + i : p.qkv, ok);
                 cp_async16_zfill(ks + tt * dkp + i, ok ? row + (p.G + g) * p.dk + i : p.qkv, ok);
                 if (MODE != SCAN_DELTA_HEAD) cp_async16_zfill(gs + tt * dkp + i, ok ? p.decay + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
-                if (MODE == SCAN_GENERAL) cp_async16_zfill(gs + (DELTA_TB + tt) * dkp + i, ok ? p.rem + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
             }
         } else {
             for (int e = threadIdx.x; e < nt * dkp; e += blockDim.x) {
@@ -419,7 +411,6 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
                 cp_async4_zfill(qs + tt * dkp + i, ok ? row + g * p.dk + i : p.qkv, ok);
                 cp_async4_zfill(ks + tt * dkp + i, ok ? row + (p.G + g) * p.dk + i : p.qkv, ok);
                 if (MODE != SCAN_DELTA_HEAD) cp_async4_zfill(gs + tt * dkp + i, ok ? p.decay + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
-                if (MODE == SCAN_GENERAL) cp_async4_zfill(gs + (DELTA_TB + tt) * dkp + i, ok ? p.rem + ((size_t)(t0 + tt) * p.H + h) * p.dk + i : p.qkv, ok);
             }
         }
         for (int e = threadIdx.x; e < nt * cols; e += blockDim.x) {
@@ -447,42 +438,10 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
         const float* qs = ds_sm + (size_t)buf * blk;
         const float* ks = qs + DELTA_TB * dkp;
         const float* gs = ks + DELTA_TB * dkp;
-        const float* vs = qs + NA * DELTA_TB * dkp;
+        const float* vs = gs + DELTA_TB * dkp;
         const float* bs = vs + DELTA_TB * cols;
         for (int tt = 0; tt < nt; tt++) {
             float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
-            if (MODE == SCAN_GENERAL) {
-                const float* es = gs + DELTA_TB * dkp;   // removal vectors
-                const float v = vs[tt * cols + jl];
-                float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
-#pragma unroll
-                for (int r4 = 0; r4 < NR / 4; r4++) {
-                    const int i = (r4 * LPC + s) * 4;
-                    const float4 k4 = *reinterpret_cast<const float4*>(ks + tt * dkp + i);
-                    const float4 g4 = *reinterpret_cast<const float4*>(gs + tt * dkp + i);
-                    const float4 q4 = *reinterpret_cast<const float4*>(qs + tt * dkp + i);
-                    r0 = fmaf(S[4 * r4], k4.x, r0); r1 = fmaf(S[4 * r4 + 1], k4.y, r1);
-                    r2 = fmaf(S[4 * r4 + 2], k4.z, r2); r3 = fmaf(S[4 * r4 + 3], k4.w, r3);
-                    S[4 * r4] += fmaf(-S[4 * r4], g4.x, k4.x * v); S[4 * r4 + 1] += fmaf(-S[4 * r4 + 1], g4.y, k4.y * v);
-                    S[4 * r4 + 2] += fmaf(-S[4 * r4 + 2], g4.z, k4.z * v); S[4 * r4 + 3] += fmaf(-S[4 * r4 + 3], g4.w, k4.w * v);
-                    o0 = fmaf(S[4 * r4], q4.x, o0); o1 = fmaf(S[4 * r4 + 1], q4.y, o1);
-                    o2 = fmaf(S[4 * r4 + 2], q4.z, o2); o3 = fmaf(S[4 * r4 + 3], q4.w, o3);
-                }
-                float held = (r0 + r1) + (r2 + r3), om = (o0 + o1) + (o2 + o3);
-#pragma unroll
-                for (int o = LPC >> 1; o > 0; o >>= 1) {
-                    held += __shfl_xor_sync(0xffffffffu, held, o);
-                    om += __shfl_xor_sync(0xffffffffu, om, o);
-                }
-#pragma unroll
-                for (int r4 = 0; r4 < NR / 4; r4++) {
-                    const float4 e4 = *reinterpret_cast<const float4*>(es + tt * dkp + (r4 * LPC + s) * 4);
-                    S[4 * r4] = fmaf(-held, e4.x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held, e4.y, S[4 * r4 + 1]);
-                    S[4 * r4 + 2] = fmaf(-held, e4.z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held, e4.w, S[4 * r4 + 3]);
-                }
-                if (s == 0 && col_ok) p.out[(size_t)(t0 + tt) * p.H * p.dv + (size_t)h * p.dv + j] = fmaf(-held, bs[tt], om);
-                continue;
-            }
             if (MODE == SCAN_PLAIN) {
                 const float u = vs[tt * cols + jl];
 #pragma unroll
@@ -541,46 +500,272 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
 // ---- generalized delta rule ---------------------------------------------------------------------------------------------------
 // The projected row is [r (H*d) | k (H*d) | v (H*d) | gate logits (H*d) | removal logits (H*d) | decay latent]; z holds the decay
 // logits (second half of the low-rank projection, bias added).  Per token, head and key channel
-//     decay = exp(-decay_rate * sigmoid(z)), kept as the loss 1 - decay          removal rate a = sigmoid(removal logit + bias)
-// and with u = k / sqrt(sum k^2 + 1e-6) the state update S <- diag(decay) S - (a u)(u^T S) + k v^T is what delta_scan_kernel's
-// SCAN_GENERAL does with b = a k / (sum k^2 + 1e-6) as the removal vector and s = S^T k.  Also the scalar r . b.  One warp per
-// (token, head); losses replace the logits in place.
+//     w = exp(-decay_rate * sigmoid(z))        a = sigmoid(removal logit + bias)        b = a k / (sum k^2 + 1e-6)
+//     S <- diag(w) S - b (S^T k)^T + k v^T,    o = S^T r                      (b (S^T k)^T is (a u)(u^T S) with u = k / |k|)
+// w enters as the loss l = 1 - w throughout: a decay a hair below one keeps its relative precision that way.
+//
+// Four tokens at a time.  With S the state before the block and P_i = w_0 .. w_{i-1} (per channel, tokens 0 .. 3 of the block),
+// everything the block reads from S is eight sums down a column,
+//     x_i = (P_i k_i)^T S,    y_i = (P_{i+1} r_i)^T S,
+// what a token's key holds follows from them and from the block's own writes,
+//     held_i = x_i + sum_{j<i} (A_ij v_j - B_ij held_j),        o_i = y_i + sum_{j<=i} (C_ij v_j - D_ij held_j),
+// with scalars per (block, head)  A_ij = sum_c k_i k_j w_{j+1} .. w_{i-1},  B_ij the same with b_j for k_j,
+// C_ij = sum_c r_i k_j w_{j+1} .. w_i,  D_ij the same with b_j; and the state after the block is
+//     S + (sum_j (k_j w_{j+1} .. w_3) v_j^T - diag(L) S) - sum_j (b_j w_{j+1} .. w_3) held_j^T,        L = 1 - w_0 w_1 w_2 w_3.
+// Only products of decays occur, no quotients.  general_delta_pre_kernel writes the block's 17 vectors [P_i k_i (4) | P_{i+1} r_i
+// (4) | k_j w.. (4) | b_j w.. (4) | L], each padded with zeros to the scan's row count, and the scalars (token i: A_i0..3, -B_i0..3,
+// C_i0..3, -D_i0..3, zeros where the sum has no term) as one contiguous record; tokens beyond the step's end are zeros, which leave
+// the state as it is.
+constexpr int GD_BLOCK = 4, GD_VECS = 17, GD_SCALARS = 64;
+inline int gd_record(int dp) { return GD_VECS * dp + GD_SCALARS; }   // floats per (block, head), dp = padded row count
 DN_DEVINL float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 DN_DEVINL float general_loss(float z, float rate) { return -expm1f(-rate * sigmoidf(z)); }
 struct GeneralDeltaPreParams {
     const float* proj; int ld;
-    float* z;                  // [T][H*d] decay logits in, losses out
+    const float* z;            // [T][H*d] decay logits
     const float* a_bias;       // [H*d]
-    float* rem; float* rb;     // [T][H*d], [T][H]
-    int T, H, d;
+    float* rec;                // [ceil(T/4)][H][record]
+    int T, H, d, dp;
     float decay_rate;
 };
+// where value `lane` of the reduced scalars goes in the record: A (6), B (6), C (10), D (10) as token * 16 + 4 * kind + j
+__device__ static const unsigned char gd_scalar_at[32] = {16, 32, 33, 48, 49, 50, 20, 36, 37, 52, 53, 54, 8, 24, 25, 40,
+                                                          41, 42, 56, 57, 58, 59, 12, 28, 29, 44, 45, 46, 60, 61, 62, 63};
 static __global__ void __launch_bounds__(128) general_delta_pre_kernel(const GeneralDeltaPreParams p) {
     pdl_launch();
     pdl_wait();
     const int lane = threadIdx.x & 31, id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (id >= p.T * p.H) return;
-    const int t = id / p.H, h = id - t * p.H, n = p.H * p.d;
-    const float* row = p.proj + (size_t)t * p.ld + (size_t)h * p.d;
-    float ss = 0.0f;
-    for (int i = lane; i < p.d; i += 32) { const float k = row[n + i]; ss += k * k; }
-    const float inv2 = 1.0f / (warp_sum(ss) + 1e-6f);
-    float rb = 0.0f;
-    const size_t o = (size_t)t * n + (size_t)h * p.d;
-    for (int i = lane; i < p.d; i += 32) {
-        const float b = sigmoidf(row[4 * n + i] + p.a_bias[(size_t)h * p.d + i]) * row[n + i] * inv2;
-        rb = fmaf(row[i], b, rb);
-        p.rem[o + i] = b;
-        p.z[o + i] = general_loss(p.z[o + i], p.decay_rate);
+    if (id >= (p.T + GD_BLOCK - 1) / GD_BLOCK * p.H) return;   // one warp per (block, head)
+    const int blk = id / p.H, h = id - blk * p.H, n = p.H * p.d, t0 = blk * GD_BLOCK;
+    const float* row = p.proj + (size_t)t0 * p.ld + (size_t)h * p.d;
+    float inv2[GD_BLOCK];
+#pragma unroll
+    for (int i = 0; i < GD_BLOCK; i++) inv2[i] = 0.0f;
+    for (int c = lane; c < p.d; c += 32)
+#pragma unroll
+        for (int i = 0; i < GD_BLOCK; i++)
+            if (t0 + i < p.T) { const float k = row[(size_t)i * p.ld + n + c]; inv2[i] += k * k; }
+#pragma unroll
+    for (int i = 0; i < GD_BLOCK; i++) inv2[i] = 1.0f / (warp_sum(inv2[i]) + 1e-6f);
+    float* rec = p.rec + (size_t)id * (GD_VECS * p.dp + GD_SCALARS);
+    float sc[32];
+#pragma unroll
+    for (int i = 0; i < 32; i++) sc[i] = 0.0f;
+    for (int c = lane; c < p.dp; c += 32) {
+        float k[4], r[4], b[4], l[4], w[4];
+#pragma unroll
+        for (int i = 0; i < GD_BLOCK; i++) {
+            k[i] = r[i] = b[i] = l[i] = 0.0f;
+            if (c < p.d && t0 + i < p.T) {
+                const float* q = row + (size_t)i * p.ld + c;
+                r[i] = q[0];
+                k[i] = q[n];
+                b[i] = sigmoidf(q[4 * (size_t)n] + p.a_bias[(size_t)h * p.d + c]) * k[i] * inv2[i];
+                l[i] = general_loss(p.z[(size_t)(t0 + i) * n + (size_t)h * p.d + c], p.decay_rate);
+            }
+            w[i] = 1.0f - l[i];
+        }
+        const float w01 = w[0] * w[1], w012 = w01 * w[2], w12 = w[1] * w[2], w23 = w[2] * w[3], w123 = w12 * w[3];
+        float* o = rec + c;
+        o[0] = k[0]; o[p.dp] = k[1] * w[0]; o[2 * p.dp] = k[2] * w01; o[3 * p.dp] = k[3] * w012;
+        o[4 * p.dp] = r[0] * w[0]; o[5 * p.dp] = r[1] * w01; o[6 * p.dp] = r[2] * w012; o[7 * p.dp] = r[3] * (w012 * w[3]);
+        o[8 * p.dp] = k[0] * w123; o[9 * p.dp] = k[1] * w23; o[10 * p.dp] = k[2] * w[3]; o[11 * p.dp] = k[3];
+        o[12 * p.dp] = b[0] * w123; o[13 * p.dp] = b[1] * w23; o[14 * p.dp] = b[2] * w[3]; o[15 * p.dp] = b[3];
+        float L = l[0];
+#pragma unroll
+        for (int i = 1; i < GD_BLOCK; i++) L = fmaf(l[i], 1.0f - L, L);
+        o[16 * p.dp] = L;
+        auto sums = [&](int at, const float (&u)[4]) {   // k_i . u_j for j < i, then r_i . u_j for j <= i, decayed in between
+            sc[at] = fmaf(k[1], u[0], sc[at]);
+            sc[at + 1] = fmaf(k[2] * w[1], u[0], sc[at + 1]); sc[at + 2] = fmaf(k[2], u[1], sc[at + 2]);
+            sc[at + 3] = fmaf(k[3] * w12, u[0], sc[at + 3]); sc[at + 4] = fmaf(k[3] * w[2], u[1], sc[at + 4]); sc[at + 5] = fmaf(k[3], u[2], sc[at + 5]);
+            const int ro = at == 0 ? 12 : 22;
+            sc[ro] = fmaf(r[0], u[0], sc[ro]);
+            sc[ro + 1] = fmaf(r[1] * w[1], u[0], sc[ro + 1]); sc[ro + 2] = fmaf(r[1], u[1], sc[ro + 2]);
+            sc[ro + 3] = fmaf(r[2] * w12, u[0], sc[ro + 3]); sc[ro + 4] = fmaf(r[2] * w[2], u[1], sc[ro + 4]); sc[ro + 5] = fmaf(r[2], u[2], sc[ro + 5]);
+            sc[ro + 6] = fmaf(r[3] * w123, u[0], sc[ro + 6]); sc[ro + 7] = fmaf(r[3] * w23, u[1], sc[ro + 7]);
+            sc[ro + 8] = fmaf(r[3] * w[3], u[2], sc[ro + 8]); sc[ro + 9] = fmaf(r[3], u[3], sc[ro + 9]);
+        };
+        sums(0, k);
+        sums(6, b);
     }
-    rb = warp_sum(rb);
-    if (lane == 0) p.rb[(size_t)t * p.H + h] = rb;
+    // 32 sums over 32 lanes: every round halves the values a lane keeps; lane i ends with sum i
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) {
+        const bool up = (lane & m) != 0;
+#pragma unroll
+        for (int i = 0; i < m; i++) {
+            const float keep = up ? sc[i + m] : sc[i], send = up ? sc[i] : sc[i + m];
+            sc[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+    }
+    float* so = rec + GD_VECS * p.dp;
+    so[lane] = 0.0f;
+    so[lane + 32] = 0.0f;
+    __syncwarp();
+    so[gd_scalar_at[lane]] = ((lane >= 6 && lane < 12) || lane >= 22) ? -sc[0] : sc[0];
+}
+
+// The scan.  Threads own state columns as in delta_scan_kernel (LPC adjacent lanes per column, NR rows each); LPC is at least 8 so
+// that the eight sums of a block can be reduced by halving: three exchange rounds leave each eighth of the lanes with one sum, the
+// rest is an ordinary reduction, and the four x_i go back to all lanes.  The lanes that hold y_i finish o_i and store it.  Records
+// arrive GD_GROUP blocks per stage through a ring of GD_RING cp.async stages.  The order of every sum is fixed.  The state is read
+// at the start (zeros when the step starts at position 0) and written back at the end.
+constexpr int GD_THREADS = 128, GD_RING = 4;
+struct GeneralDeltaScanParams {
+    const float* rec;          // [ceil(T/4)][H][record]
+    const float* v; int ld;    // values of token t, head h at v + t * ld + h * d
+    float* state;              // [H][d][d]
+    float* out;                // [T][H*d]
+    int T, H, d;
+    PosSrc ps;
+};
+template <int NR, int LPC> __host__ __device__ constexpr int gd_group() { return NR * LPC > 256 ? 1 : 2; }
+template <int NR, int LPC> inline size_t general_delta_scan_smem() {
+    return (size_t)GD_RING * gd_group<NR, LPC>() * (GD_VECS * NR * LPC + GD_SCALARS + GD_BLOCK * (GD_THREADS / LPC)) * 4;
+}
+template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general_delta_scan_kernel(const GeneralDeltaScanParams p) {
+    extern __shared__ __align__(16) float gs_sm[];
+    pdl_launch();
+    pdl_wait();
+    static_assert(NR % 4 == 0 && LPC >= 8 && LPC <= 32, "scan shape");
+    constexpr int cols = GD_THREADS / LPC, dp = NR * LPC, REC = GD_VECS * dp + GD_SCALARS, GROUP = gd_group<NR, LPC>();
+    constexpr int blk_fl = REC + GD_BLOCK * cols, stage_fl = GROUP * blk_fl;
+    const int h = blockIdx.y;
+    const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC, j = blockIdx.x * cols + jl;
+    const bool col_ok = j < p.d;
+    const uint32_t pos0 = pos_of(p.ps);
+    const int n_blk = (p.T + GD_BLOCK - 1) / GD_BLOCK, n_stage = (n_blk + GROUP - 1) / GROUP;
+    auto stage = [&](int st) {
+        if (st < n_stage) {
+#pragma unroll
+            for (int g = 0; g < GROUP; g++) {
+                const int b = st * GROUP + g;
+                float* dst = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
+                if (b < n_blk) {
+                    const float* src = p.rec + ((size_t)b * p.H + h) * REC;
+                    for (int e = threadIdx.x; e < REC / 4; e += GD_THREADS) cp_async16_zfill(dst + 4 * e, src + 4 * e, true);
+                    for (int e = threadIdx.x; e < GD_BLOCK * cols; e += GD_THREADS) {
+                        const int c = e >> 2, i = e & 3, t = b * GD_BLOCK + i, jj = blockIdx.x * cols + c;   // [column][token]
+                        const bool ok = t < p.T && jj < p.d;
+                        cp_async4_zfill(dst + REC + e, ok ? p.v + (size_t)t * p.ld + (size_t)h * p.d + jj : p.v, ok);
+                    }
+                }
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int st = 0; st < GD_RING - 1; st++) stage(st);
+    float S[NR];
+    float* sp = p.state + ((size_t)h * p.d) * p.d + j;
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
+        S[r] = (pos0 > 0 && col_ok && i < p.d) ? sp[(size_t)i * p.d] : 0.0f;
+    }
+    const int which = s / (LPC / 8);   // the sum this lane ends with: 0 .. 3 x_i, 4 .. 7 y_i
+    float* outp = p.out + (size_t)h * p.d + j;
+    for (int st = 0; st < n_stage; st++) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
+        __syncthreads();   // this stage has landed for everyone, and everyone is done with the one that is overwritten next
+        stage(st + GD_RING - 1);
+#pragma unroll
+        for (int g = 0; g < GROUP; g++) {
+            const int b = st * GROUP + g;
+            if (b >= n_blk) break;
+            const float* rec = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
+            const float4 v4 = *reinterpret_cast<const float4*>(rec + REC + 4 * jl);
+            float d[8];
+#pragma unroll
+            for (int q = 0; q < 8; q++) d[q] = 0.0f;
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) {
+                const int i = (r4 * LPC + s) * 4;
+#pragma unroll
+                for (int q = 0; q < 8; q++) {
+                    const float4 a = *reinterpret_cast<const float4*>(rec + q * dp + i);
+                    d[q] = fmaf(S[4 * r4], a.x, d[q]); d[q] = fmaf(S[4 * r4 + 1], a.y, d[q]);
+                    d[q] = fmaf(S[4 * r4 + 2], a.z, d[q]); d[q] = fmaf(S[4 * r4 + 3], a.w, d[q]);
+                }
+            }
+            // decay and writes: nothing here waits for the reductions
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) {
+                const int i = (r4 * LPC + s) * 4;
+                float4 u = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                for (int q = 0; q < 4; q++) {
+                    const float4 a = *reinterpret_cast<const float4*>(rec + (8 + q) * dp + i);
+                    const float v = q == 0 ? v4.x : q == 1 ? v4.y : q == 2 ? v4.z : v4.w;
+                    u.x = fmaf(a.x, v, u.x); u.y = fmaf(a.y, v, u.y); u.z = fmaf(a.z, v, u.z); u.w = fmaf(a.w, v, u.w);
+                }
+                const float4 L = *reinterpret_cast<const float4*>(rec + 16 * dp + i);
+                S[4 * r4] += fmaf(-L.x, S[4 * r4], u.x); S[4 * r4 + 1] += fmaf(-L.y, S[4 * r4 + 1], u.y);
+                S[4 * r4 + 2] += fmaf(-L.z, S[4 * r4 + 2], u.z); S[4 * r4 + 3] += fmaf(-L.w, S[4 * r4 + 3], u.w);
+            }
+            // eight sums over LPC lanes by halving
+#pragma unroll
+            for (int m = 4; m > 0; m >>= 1) {
+                const int lm = m * (LPC / 8);
+                const bool up = (s & lm) != 0;
+#pragma unroll
+                for (int q = 0; q < m; q++) {
+                    const float keep = up ? d[q + m] : d[q], send = up ? d[q] : d[q + m];
+                    d[q] = keep + __shfl_xor_sync(0xffffffffu, send, lm);
+                }
+            }
+#pragma unroll
+            for (int lm = LPC / 16; lm > 0; lm >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], lm);
+            const float* sc = rec + GD_VECS * dp;
+            float held[4];
+#pragma unroll
+            for (int q = 0; q < 4; q++) held[q] = __shfl_sync(0xffffffffu, d[0], q * (LPC / 8), LPC);
+            {
+                const float4 a1 = *reinterpret_cast<const float4*>(sc + 16), b1 = *reinterpret_cast<const float4*>(sc + 20);
+                const float4 a2 = *reinterpret_cast<const float4*>(sc + 32), b2 = *reinterpret_cast<const float4*>(sc + 36);
+                const float4 a3 = *reinterpret_cast<const float4*>(sc + 48), b3 = *reinterpret_cast<const float4*>(sc + 52);
+                held[1] = fmaf(b1.x, held[0], fmaf(a1.x, v4.x, held[1]));
+                held[2] = fmaf(b2.x, held[0], fmaf(a2.y, v4.y, fmaf(a2.x, v4.x, held[2])));
+                held[2] = fmaf(b2.y, held[1], held[2]);
+                held[3] = fmaf(b3.x, held[0], fmaf(a3.z, v4.z, fmaf(a3.y, v4.y, fmaf(a3.x, v4.x, held[3]))));
+                held[3] = fmaf(b3.z, held[2], fmaf(b3.y, held[1], held[3]));
+            }
+            // removals
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) {
+                const int i = (r4 * LPC + s) * 4;
+#pragma unroll
+                for (int q = 0; q < 4; q++) {
+                    const float4 e = *reinterpret_cast<const float4*>(rec + (12 + q) * dp + i);
+                    S[4 * r4] = fmaf(-held[q], e.x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held[q], e.y, S[4 * r4 + 1]);
+                    S[4 * r4 + 2] = fmaf(-held[q], e.z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held[q], e.w, S[4 * r4 + 3]);
+                }
+            }
+            {
+                const int i = which & 3, t = b * GD_BLOCK + i;
+                const float4 c4 = *reinterpret_cast<const float4*>(sc + 16 * i + 8), e4 = *reinterpret_cast<const float4*>(sc + 16 * i + 12);
+                float o = fmaf(c4.x, v4.x, d[0]);
+                o = fmaf(c4.y, v4.y, o); o = fmaf(c4.z, v4.z, o); o = fmaf(c4.w, v4.w, o);
+                o = fmaf(e4.x, held[0], o); o = fmaf(e4.y, held[1], o); o = fmaf(e4.z, held[2], o); o = fmaf(e4.w, held[3], o);
+                if (which >= 4 && s % (LPC / 8) == 0 && col_ok && t < p.T) outp[(size_t)t * p.H * p.d] = o;
+            }
+        }
+    }
+    if (col_ok) {
+#pragma unroll
+        for (int r = 0; r < NR; r++) {
+            const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
+            if (i < p.d) sp[(size_t)i * p.d] = S[r];
+        }
+    }
 }
 
 // One token of the rule, one CTA per head: the projected row in, the operand-type row rms(o) * w * sigmoid(gate) out.  The low-rank
 // latent passes tanh and is rounded to the operand type (what the many-token path feeds its product), the second half of the
-// projection is done here.  Threads are columns x row groups; the state goes past twice (once for S^T k, once for the update and
-// the read-out), the second time from L1.  Shared memory: ra + 4 d + blockDim.x floats (+ the reduction slots).
+// projection is done here.  Threads are columns x row groups; RPT > 0: a thread's state rows (at most RPT) are loaded first of all
+// and stay in registers; 0: any size, columns in passes, the state read twice, the second time from L1.  Shared memory:
+// ra + 5 d + blockDim.x floats (+ the reduction slots).
 template <typename AT, typename WT> struct GeneralDeltaStepParams {
     const float* proj;         // the token's row; decay latent (before tanh) at column 5 * H * d
     const WT* w2; int ra;      // [H*d][ra]
@@ -591,7 +776,7 @@ template <typename AT, typename WT> struct GeneralDeltaStepParams {
     float decay_rate;
     PosSrc ps;
 };
-template <typename AT, typename WT> __global__ void __launch_bounds__(1024) general_delta_step_kernel(const GeneralDeltaStepParams<AT, WT> p) {
+template <typename AT, typename WT, int RPT> __global__ void __launch_bounds__(1024) general_delta_step_kernel(const GeneralDeltaStepParams<AT, WT> p) {
     extern __shared__ __align__(16) float gd_sm[];
     __shared__ float red[33];
     pdl_launch();
@@ -601,20 +786,42 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
     float* ks = lat + p.ra;        // [d] key
     float* ws = ks + d;            // [d] losses
     float* bs = ws + d;            // [d] removal vector
-    float* os = bs + d;            // [d] read-out
+    float* rs = bs + d;            // [d] query
+    float* os = rs + d;            // [d] read-out
     float* part = os + d;          // [blockDim.x] sums of the row groups
     const float* row = p.proj + (size_t)h * d;
+    const bool fresh = pos_of(p.ps) == 0;
+    const int c = threadIdx.x % p.cw, rg = threadIdx.x / p.cw, groups = blockDim.x / p.cw;
+    const int per = (d + groups - 1) / groups, i0 = min(d, rg * per), i1 = min(d, i0 + per);
+    float* S = p.state + (size_t)h * d * d;
+    constexpr int NREG = RPT > 0 ? RPT : 1;
+    float old[NREG];
+    if (RPT > 0) {
+#pragma unroll
+        for (int e = 0; e < NREG; e++) old[e] = i0 + e < i1 && c < d && !fresh ? S[(size_t)(i0 + e) * d + c] : 0.0f;
+    }
     for (int i = threadIdx.x; i < p.ra; i += blockDim.x) { AT v; from_f(v, tanhf(p.proj[5 * (size_t)n + i])); lat[i] = to_f(v); }
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) { const float k = row[n + i]; ks[i] = k; ss += k * k; }
+    for (int i = threadIdx.x; i < d; i += blockDim.x) { const float k = row[n + i]; ks[i] = k; rs[i] = row[i]; ss += k * k; }
     const float inv2 = 1.0f / (block_sum(ss, red) + 1e-6f);   // (its barriers also publish lat and ks)
     // decay logits: eight lanes per key channel
-    for (int i0 = 0; i0 < d; i0 += blockDim.x >> 3) {
-        const int i = i0 + (threadIdx.x >> 3), l8 = threadIdx.x & 7;
+    const bool vec = p.ra % Vec16<WT>::N == 0;
+    for (int k0 = 0; k0 < d; k0 += blockDim.x >> 3) {
+        const int i = k0 + (threadIdx.x >> 3), l8 = threadIdx.x & 7;
         float z = 0.0f;
         if (i < d) {
             const WT* w2 = p.w2 + ((size_t)h * d + i) * p.ra;
-            for (int j = l8; j < p.ra; j += 8) z = fmaf(to_f(w2[j]), lat[j], z);
+            if (vec) {
+                constexpr int N = Vec16<WT>::N;
+                for (int j = l8 * N; j < p.ra; j += 8 * N) {
+                    float v[N];
+                    load16<WT>(w2 + j, v);
+#pragma unroll
+                    for (int e = 0; e < N; e++) z = fmaf(v[e], lat[j + e], z);
+                }
+            } else {
+                for (int j = l8; j < p.ra; j += 8) z = fmaf(to_f(w2[j]), lat[j], z);
+            }
         }
         z += __shfl_xor_sync(0xffffffffu, z, 4);
         z += __shfl_xor_sync(0xffffffffu, z, 2);
@@ -625,14 +832,14 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
         }
     }
     __syncthreads();
-    const bool fresh = pos_of(p.ps) == 0;
-    const int c = threadIdx.x % p.cw, rg = threadIdx.x / p.cw, groups = blockDim.x / p.cw;
-    const int per = (d + groups - 1) / groups, i0 = min(d, rg * per), i1 = min(d, i0 + per);
-    float* S = p.state + (size_t)h * d * d;
     for (int c0 = 0; c0 < d; c0 += p.cw) {
         const int j = c0 + c;
         float held = 0.0f;
-        if (j < d && !fresh) {
+        if (RPT > 0) {
+#pragma unroll
+            for (int e = 0; e < NREG; e++)
+                if (i0 + e < i1) held = fmaf(old[e], ks[i0 + e], held);
+        } else if (j < d && !fresh) {
 #pragma unroll 8
             for (int i = i0; i < i1; i++) held = fmaf(S[(size_t)i * d + j], ks[i], held);
         }
@@ -644,20 +851,24 @@ template <typename AT, typename WT> __global__ void __launch_bounds__(1024) gene
         float o = 0.0f;
         if (j < d) {
             const float v = row[2 * (size_t)n + j];
-            for (int ib = i0; ib < i1; ib += 4) {   // four rows' loads ahead of their stores
-                float old[4], r[4];
+            auto update = [&](int i, float was) {
+                const float nw = fmaf(-bs[i], held, was + fmaf(-ws[i], was, ks[i] * v));
+                S[(size_t)i * d + j] = nw;
+                o = fmaf(nw, rs[i], o);
+            };
+            if (RPT > 0) {
 #pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    old[e] = ib + e < i1 && !fresh ? S[(size_t)(ib + e) * d + j] : 0.0f;
-                    r[e] = ib + e < i1 ? row[ib + e] : 0.0f;
+                for (int e = 0; e < NREG; e++)
+                    if (i0 + e < i1) update(i0 + e, old[e]);
+            } else {
+                for (int ib = i0; ib < i1; ib += 4) {   // four rows' loads ahead of their stores
+                    float was[4];
+#pragma unroll
+                    for (int e = 0; e < 4; e++) was[e] = ib + e < i1 && !fresh ? S[(size_t)(ib + e) * d + j] : 0.0f;
+#pragma unroll
+                    for (int e = 0; e < 4; e++)
+                        if (ib + e < i1) update(ib + e, was[e]);
                 }
-#pragma unroll
-                for (int e = 0; e < 4; e++)
-                    if (ib + e < i1) {
-                        const float nw = fmaf(-bs[ib + e], held, old[e] + fmaf(-ws[ib + e], old[e], ks[ib + e] * v));
-                        S[(size_t)(ib + e) * d + j] = nw;
-                        o = fmaf(nw, r[e], o);
-                    }
             }
         }
         part[threadIdx.x] = o;
