@@ -336,7 +336,7 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         scan_shape(c.d, &nr, &lpc);
         GeneralDeltaPreParams pp{};
         pp.proj = proj; pp.ld = L.in_rows; pp.z = z; pp.a_bias = L.a_bias; pp.rec = rec; pp.T = T; pp.H = c.H; pp.d = c.d; pp.dp = nr * lpc; pp.decay_rate = decay_rate;
-        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3(((T + GD_BLOCK - 1) / GD_BLOCK * c.H + 3) / 4), dim3(128), 0, pp)) return 1;
+        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3(c.H, (T + GD_BLOCK - 1) / GD_BLOCK), dim3(pp.dp), 0, pp)) return 1;
         GeneralDeltaScanParams sp{};
         sp.rec = rec; sp.v = proj + 2 * (size_t)n; sp.ld = L.in_rows; sp.state = L.state; sp.out = fo; sp.T = T; sp.H = c.H; sp.d = c.d; sp.ps = ps;
         if (scan(st, nr, lpc, sp)) return 1;

@@ -531,64 +531,57 @@ struct GeneralDeltaPreParams {
 // where value `lane` of the reduced scalars goes in the record: A (6), B (6), C (10), D (10) as token * 16 + 4 * kind + j
 __device__ static const unsigned char gd_scalar_at[32] = {16, 32, 33, 48, 49, 50, 20, 36, 37, 52, 53, 54, 8, 24, 25, 40,
                                                           41, 42, 56, 57, 58, 59, 12, 28, 29, 44, 45, 46, 60, 61, 62, 63};
-static __global__ void __launch_bounds__(128) general_delta_pre_kernel(const GeneralDeltaPreParams p) {
+// One CTA per (block, head), a thread per padded channel.  The
+// removal vectors stay unnormalised through the reductions -- B and D are linear in 1 / (sum k^2 + 1e-6) of token j.
+static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const GeneralDeltaPreParams p) {
+    __shared__ float part[16][36];   // per warp: the 32 sums, then the squared lengths of the four keys
     pdl_launch();
     pdl_wait();
-    const int lane = threadIdx.x & 31, id = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (id >= (p.T + GD_BLOCK - 1) / GD_BLOCK * p.H) return;   // one warp per (block, head)
-    const int blk = id / p.H, h = id - blk * p.H, n = p.H * p.d, t0 = blk * GD_BLOCK;
-    const float* row = p.proj + (size_t)t0 * p.ld + (size_t)h * p.d;
-    float inv2[GD_BLOCK];
-#pragma unroll
-    for (int i = 0; i < GD_BLOCK; i++) inv2[i] = 0.0f;
-    for (int c = lane; c < p.d; c += 32)
-#pragma unroll
-        for (int i = 0; i < GD_BLOCK; i++)
-            if (t0 + i < p.T) { const float k = row[(size_t)i * p.ld + n + c]; inv2[i] += k * k; }
-#pragma unroll
-    for (int i = 0; i < GD_BLOCK; i++) inv2[i] = 1.0f / (warp_sum(inv2[i]) + 1e-6f);
-    float* rec = p.rec + (size_t)id * (GD_VECS * p.dp + GD_SCALARS);
-    float sc[32];
-#pragma unroll
-    for (int i = 0; i < 32; i++) sc[i] = 0.0f;
-    for (int c = lane; c < p.dp; c += 32) {
-        float k[4], r[4], b[4], l[4], w[4];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, c = threadIdx.x;
+    const int blk = blockIdx.y, h = blockIdx.x, n = p.H * p.d, t0 = blk * GD_BLOCK;
+    float* rec = p.rec + ((size_t)blk * p.H + h) * (GD_VECS * p.dp + GD_SCALARS);
+    float k[4], r[4], b[4], l[4], w[4];
+    {
+        float za[4], aa[4];
+        const float* q = p.proj + (size_t)t0 * p.ld + (size_t)h * p.d + c;
+        const float* zp = p.z + (size_t)t0 * n + (size_t)h * p.d + c;
 #pragma unroll
         for (int i = 0; i < GD_BLOCK; i++) {
-            k[i] = r[i] = b[i] = l[i] = 0.0f;
-            if (c < p.d && t0 + i < p.T) {
-                const float* q = row + (size_t)i * p.ld + c;
-                r[i] = q[0];
-                k[i] = q[n];
-                b[i] = sigmoidf(q[4 * (size_t)n] + p.a_bias[(size_t)h * p.d + c]) * k[i] * inv2[i];
-                l[i] = general_loss(p.z[(size_t)(t0 + i) * n + (size_t)h * p.d + c], p.decay_rate);
-            }
+            const bool ok = c < p.d && t0 + i < p.T;
+            r[i] = ok ? q[(size_t)i * p.ld] : 0.0f;
+            k[i] = ok ? q[(size_t)i * p.ld + n] : 0.0f;
+            aa[i] = ok ? q[(size_t)i * p.ld + 4 * (size_t)n] : 0.0f;
+            za[i] = ok ? zp[(size_t)i * n] : 0.0f;
+        }
+        const float ab = c < p.d ? p.a_bias[(size_t)h * p.d + c] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < GD_BLOCK; i++) {
+            b[i] = sigmoidf(aa[i] + ab) * k[i];
+            l[i] = c < p.d && t0 + i < p.T ? general_loss(za[i], p.decay_rate) : 0.0f;
             w[i] = 1.0f - l[i];
         }
-        const float w01 = w[0] * w[1], w012 = w01 * w[2], w12 = w[1] * w[2], w23 = w[2] * w[3], w123 = w12 * w[3];
-        float* o = rec + c;
-        o[0] = k[0]; o[p.dp] = k[1] * w[0]; o[2 * p.dp] = k[2] * w01; o[3 * p.dp] = k[3] * w012;
-        o[4 * p.dp] = r[0] * w[0]; o[5 * p.dp] = r[1] * w01; o[6 * p.dp] = r[2] * w012; o[7 * p.dp] = r[3] * (w012 * w[3]);
-        o[8 * p.dp] = k[0] * w123; o[9 * p.dp] = k[1] * w23; o[10 * p.dp] = k[2] * w[3]; o[11 * p.dp] = k[3];
-        o[12 * p.dp] = b[0] * w123; o[13 * p.dp] = b[1] * w23; o[14 * p.dp] = b[2] * w[3]; o[15 * p.dp] = b[3];
-        float L = l[0];
-#pragma unroll
-        for (int i = 1; i < GD_BLOCK; i++) L = fmaf(l[i], 1.0f - L, L);
-        o[16 * p.dp] = L;
-        auto sums = [&](int at, const float (&u)[4]) {   // k_i . u_j for j < i, then r_i . u_j for j <= i, decayed in between
-            sc[at] = fmaf(k[1], u[0], sc[at]);
-            sc[at + 1] = fmaf(k[2] * w[1], u[0], sc[at + 1]); sc[at + 2] = fmaf(k[2], u[1], sc[at + 2]);
-            sc[at + 3] = fmaf(k[3] * w12, u[0], sc[at + 3]); sc[at + 4] = fmaf(k[3] * w[2], u[1], sc[at + 4]); sc[at + 5] = fmaf(k[3], u[2], sc[at + 5]);
-            const int ro = at == 0 ? 12 : 22;
-            sc[ro] = fmaf(r[0], u[0], sc[ro]);
-            sc[ro + 1] = fmaf(r[1] * w[1], u[0], sc[ro + 1]); sc[ro + 2] = fmaf(r[1], u[1], sc[ro + 2]);
-            sc[ro + 3] = fmaf(r[2] * w12, u[0], sc[ro + 3]); sc[ro + 4] = fmaf(r[2] * w[2], u[1], sc[ro + 4]); sc[ro + 5] = fmaf(r[2], u[2], sc[ro + 5]);
-            sc[ro + 6] = fmaf(r[3] * w123, u[0], sc[ro + 6]); sc[ro + 7] = fmaf(r[3] * w23, u[1], sc[ro + 7]);
-            sc[ro + 8] = fmaf(r[3] * w[3], u[2], sc[ro + 8]); sc[ro + 9] = fmaf(r[3], u[3], sc[ro + 9]);
-        };
-        sums(0, k);
-        sums(6, b);
     }
+    const float w01 = w[0] * w[1], w012 = w01 * w[2], w12 = w[1] * w[2], w23 = w[2] * w[3], w123 = w12 * w[3];
+    float* o = rec + c;
+    o[0] = k[0]; o[p.dp] = k[1] * w[0]; o[2 * p.dp] = k[2] * w01; o[3 * p.dp] = k[3] * w012;
+    o[4 * p.dp] = r[0] * w[0]; o[5 * p.dp] = r[1] * w01; o[6 * p.dp] = r[2] * w012; o[7 * p.dp] = r[3] * (w012 * w[3]);
+    o[8 * p.dp] = k[0] * w123; o[9 * p.dp] = k[1] * w23; o[10 * p.dp] = k[2] * w[3]; o[11 * p.dp] = k[3];
+    float L = l[0];
+#pragma unroll
+    for (int i = 1; i < GD_BLOCK; i++) L = fmaf(l[i], 1.0f - L, L);
+    o[16 * p.dp] = L;
+    float sc[32];
+    auto sums = [&](int at, int ro, const float (&u)[4]) {   // k_i . u_j for j < i, then r_i . u_j for j <= i, decayed in between
+        sc[at] = k[1] * u[0];
+        sc[at + 1] = k[2] * w[1] * u[0]; sc[at + 2] = k[2] * u[1];
+        sc[at + 3] = k[3] * w12 * u[0]; sc[at + 4] = k[3] * w[2] * u[1]; sc[at + 5] = k[3] * u[2];
+        sc[ro] = r[0] * u[0];
+        sc[ro + 1] = r[1] * w[1] * u[0]; sc[ro + 2] = r[1] * u[1];
+        sc[ro + 3] = r[2] * w12 * u[0]; sc[ro + 4] = r[2] * w[2] * u[1]; sc[ro + 5] = r[2] * u[2];
+        sc[ro + 6] = r[3] * w123 * u[0]; sc[ro + 7] = r[3] * w23 * u[1]; sc[ro + 8] = r[3] * w[3] * u[2]; sc[ro + 9] = r[3] * u[3];
+    };
+    sums(0, 12, k);
+    sums(6, 22, b);
     // 32 sums over 32 lanes: every round halves the values a lane keeps; lane i ends with sum i
 #pragma unroll
     for (int m = 16; m > 0; m >>= 1) {
@@ -599,11 +592,42 @@ static __global__ void __launch_bounds__(128) general_delta_pre_kernel(const Gen
             sc[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
         }
     }
-    float* so = rec + GD_VECS * p.dp;
-    so[lane] = 0.0f;
-    so[lane + 32] = 0.0f;
-    __syncwarp();
-    so[gd_scalar_at[lane]] = ((lane >= 6 && lane < 12) || lane >= 22) ? -sc[0] : sc[0];
+    float kk[4];
+#pragma unroll
+    for (int i = 0; i < GD_BLOCK; i++) kk[i] = k[i] * k[i];
+#pragma unroll
+    for (int m = 2; m > 0; m >>= 1) {
+        const bool up = (lane & (8 * m)) != 0;
+#pragma unroll
+        for (int i = 0; i < m; i++) {
+            const float keep = up ? kk[i + m] : kk[i], send = up ? kk[i] : kk[i + m];
+            kk[i] = keep + __shfl_xor_sync(0xffffffffu, send, 8 * m);
+        }
+    }
+#pragma unroll
+    for (int m = 4; m > 0; m >>= 1) kk[0] += __shfl_xor_sync(0xffffffffu, kk[0], m);
+    part[warp][lane] = sc[0];
+    if ((lane & 7) == 0) part[warp][32 + (lane >> 3)] = kk[0];
+    __syncthreads();
+    float inv2[4];
+#pragma unroll
+    for (int i = 0; i < GD_BLOCK; i++) {
+        float s = 0.0f;
+        for (int g = 0; g < n_warps; g++) s += part[g][32 + i];
+        inv2[i] = 1.0f / (s + 1e-6f);
+    }
+    o[12 * p.dp] = b[0] * inv2[0] * w123; o[13 * p.dp] = b[1] * inv2[1] * w23; o[14 * p.dp] = b[2] * inv2[2] * w[3]; o[15 * p.dp] = b[3] * inv2[3];
+    if (warp == 0) {
+        float s = 0.0f;
+        for (int g = 0; g < n_warps; g++) s += part[g][lane];
+        const int at = gd_scalar_at[lane];
+        if (at & 4) s *= -((at & 3) == 0 ? inv2[0] : (at & 3) == 1 ? inv2[1] : (at & 3) == 2 ? inv2[2] : inv2[3]);   // B, D: removal of token j
+        float* so = rec + GD_VECS * p.dp;
+        so[lane] = 0.0f;
+        so[lane + 32] = 0.0f;
+        __syncwarp();
+        so[at] = s;
+    }
 }
 
 // The scan.  Threads own state columns as in delta_scan_kernel (LPC adjacent lanes per column, NR rows each); LPC is at least 8 so
@@ -641,15 +665,14 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
 #pragma unroll
             for (int g = 0; g < GROUP; g++) {
                 const int b = st * GROUP + g;
+                const bool real = b < n_blk;   // a block beyond the end is zeros: it leaves the state as it is
                 float* dst = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
-                if (b < n_blk) {
-                    const float* src = p.rec + ((size_t)b * p.H + h) * REC;
-                    for (int e = threadIdx.x; e < REC / 4; e += GD_THREADS) cp_async16_zfill(dst + 4 * e, src + 4 * e, true);
-                    for (int e = threadIdx.x; e < GD_BLOCK * cols; e += GD_THREADS) {
-                        const int c = e >> 2, i = e & 3, t = b * GD_BLOCK + i, jj = blockIdx.x * cols + c;   // [column][token]
-                        const bool ok = t < p.T && jj < p.d;
-                        cp_async4_zfill(dst + REC + e, ok ? p.v + (size_t)t * p.ld + (size_t)h * p.d + jj : p.v, ok);
-                    }
+                const float* src = p.rec + ((size_t)(real ? b : 0) * p.H + h) * REC;
+                for (int e = threadIdx.x; e < REC / 4; e += GD_THREADS) cp_async16_zfill(dst + 4 * e, src + 4 * e, real);
+                for (int e = threadIdx.x; e < GD_BLOCK * cols; e += GD_THREADS) {
+                    const int c = e >> 2, i = e & 3, t = b * GD_BLOCK + i, jj = blockIdx.x * cols + c;   // [column][token]
+                    const bool ok = t < p.T && jj < p.d;
+                    cp_async4_zfill(dst + REC + e, ok ? p.v + (size_t)t * p.ld + (size_t)h * p.d + jj : p.v, ok);
                 }
             }
         }
@@ -665,91 +688,109 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
         S[r] = (pos0 > 0 && col_ok && i < p.d) ? sp[(size_t)i * p.d] : 0.0f;
     }
     const int which = s / (LPC / 8);   // the sum this lane ends with: 0 .. 3 x_i, 4 .. 7 y_i
-    float* outp = p.out + (size_t)h * p.d + j;
+    const int oi = which & 3;          // ... and the token of the block it finishes when it is y_i
+    const bool stores = which >= 4 && s % (LPC / 8) == 0 && col_ok;
+    float* outp = p.out + (size_t)oi * p.H * p.d + (size_t)h * p.d + j;
+    // a block's dot vectors and values are read into registers while the block before it is being reduced
+    float4 nx[8][NR / 4], nv;
+    auto fetch = [&](const float* rec) {
+#pragma unroll
+        for (int q = 0; q < 8; q++)
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) nx[q][r4] = *reinterpret_cast<const float4*>(rec + q * dp + (r4 * LPC + s) * 4);
+        nv = *reinterpret_cast<const float4*>(rec + REC + 4 * jl);
+    };
+    asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
+    __syncthreads();
+    fetch(gs_sm);
     for (int st = 0; st < n_stage; st++) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
-        __syncthreads();   // this stage has landed for everyone, and everyone is done with the one that is overwritten next
-        stage(st + GD_RING - 1);
+        stage(st + GD_RING - 1);   // into the place of stage st - 1, which everyone has read
 #pragma unroll
         for (int g = 0; g < GROUP; g++) {
-            const int b = st * GROUP + g;
-            if (b >= n_blk) break;
             const float* rec = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
-            const float4 v4 = *reinterpret_cast<const float4*>(rec + REC + 4 * jl);
+            const float* sc = rec + GD_VECS * dp;
+            const float4 v4 = nv;
+            float4 kv[4][NR / 4], bv[4][NR / 4], Lv[NR / 4];
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) {
+#pragma unroll
+                for (int q = 0; q < 4; q++) kv[q][r4] = *reinterpret_cast<const float4*>(rec + (8 + q) * dp + (r4 * LPC + s) * 4);
+                Lv[r4] = *reinterpret_cast<const float4*>(rec + 16 * dp + (r4 * LPC + s) * 4);
+            }
+            const float4 a1 = *reinterpret_cast<const float4*>(sc + 16), b1 = *reinterpret_cast<const float4*>(sc + 20);
+            const float4 a2 = *reinterpret_cast<const float4*>(sc + 32), b2 = *reinterpret_cast<const float4*>(sc + 36);
+            const float4 a3 = *reinterpret_cast<const float4*>(sc + 48), b3 = *reinterpret_cast<const float4*>(sc + 52);
+            const float4 c4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 8), e4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 12);
             float d[8];
 #pragma unroll
             for (int q = 0; q < 8; q++) d[q] = 0.0f;
 #pragma unroll
             for (int r4 = 0; r4 < NR / 4; r4++) {
-                const int i = (r4 * LPC + s) * 4;
 #pragma unroll
-                for (int q = 0; q < 8; q++) {
-                    const float4 a = *reinterpret_cast<const float4*>(rec + q * dp + i);
-                    d[q] = fmaf(S[4 * r4], a.x, d[q]); d[q] = fmaf(S[4 * r4 + 1], a.y, d[q]);
-                    d[q] = fmaf(S[4 * r4 + 2], a.z, d[q]); d[q] = fmaf(S[4 * r4 + 3], a.w, d[q]);
-                }
+                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4], nx[q][r4].x, d[q]);
+#pragma unroll
+                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 1], nx[q][r4].y, d[q]);
+#pragma unroll
+                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 2], nx[q][r4].z, d[q]);
+#pragma unroll
+                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 3], nx[q][r4].w, d[q]);
             }
-            // decay and writes: nothing here waits for the reductions
-#pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) {
-                const int i = (r4 * LPC + s) * 4;
-                float4 u = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll
-                for (int q = 0; q < 4; q++) {
-                    const float4 a = *reinterpret_cast<const float4*>(rec + (8 + q) * dp + i);
-                    const float v = q == 0 ? v4.x : q == 1 ? v4.y : q == 2 ? v4.z : v4.w;
-                    u.x = fmaf(a.x, v, u.x); u.y = fmaf(a.y, v, u.y); u.z = fmaf(a.z, v, u.z); u.w = fmaf(a.w, v, u.w);
-                }
-                const float4 L = *reinterpret_cast<const float4*>(rec + 16 * dp + i);
-                S[4 * r4] += fmaf(-L.x, S[4 * r4], u.x); S[4 * r4 + 1] += fmaf(-L.y, S[4 * r4 + 1], u.y);
-                S[4 * r4 + 2] += fmaf(-L.z, S[4 * r4 + 2], u.z); S[4 * r4 + 3] += fmaf(-L.w, S[4 * r4 + 3], u.w);
-            }
-            // eight sums over LPC lanes by halving
-#pragma unroll
-            for (int m = 4; m > 0; m >>= 1) {
+            // first exchange of the reduction (eight sums over LPC lanes by halving)
+            auto halve = [&](int m) {
                 const int lm = m * (LPC / 8);
                 const bool up = (s & lm) != 0;
 #pragma unroll
-                for (int q = 0; q < m; q++) {
-                    const float keep = up ? d[q + m] : d[q], send = up ? d[q] : d[q + m];
-                    d[q] = keep + __shfl_xor_sync(0xffffffffu, send, lm);
-                }
+                for (int q = 0; q < 4; q++)
+                    if (q < m) {
+                        const float keep = up ? d[q + m] : d[q], send = up ? d[q] : d[q + m];
+                        d[q] = keep + __shfl_xor_sync(0xffffffffu, send, lm);
+                    }
+            };
+            halve(4);
+            // decay and writes: nothing here waits for the reduction
+#pragma unroll
+            for (int r4 = 0; r4 < NR / 4; r4++) {
+                auto write = [&](float& x, float L, float k0, float k1, float k2, float k3) {
+                    x += fmaf(-L, x, fmaf(k3, v4.w, fmaf(k2, v4.z, fmaf(k1, v4.y, k0 * v4.x))));
+                };
+                write(S[4 * r4], Lv[r4].x, kv[0][r4].x, kv[1][r4].x, kv[2][r4].x, kv[3][r4].x);
+                write(S[4 * r4 + 1], Lv[r4].y, kv[0][r4].y, kv[1][r4].y, kv[2][r4].y, kv[3][r4].y);
+                write(S[4 * r4 + 2], Lv[r4].z, kv[0][r4].z, kv[1][r4].z, kv[2][r4].z, kv[3][r4].z);
+                write(S[4 * r4 + 3], Lv[r4].w, kv[0][r4].w, kv[1][r4].w, kv[2][r4].w, kv[3][r4].w);
+#pragma unroll
+                for (int q = 0; q < 4; q++) bv[q][r4] = *reinterpret_cast<const float4*>(rec + (12 + q) * dp + (r4 * LPC + s) * 4);
             }
+            halve(2);
+            if (g + 1 < GROUP) {
+                fetch(rec + blk_fl);
+            } else if (st + 1 < n_stage) {
+                asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
+                __syncthreads();   // the next stage has landed for everyone, and everyone has read this one
+                fetch(gs_sm + (size_t)((st + 1) % GD_RING) * stage_fl);
+            }
+            halve(1);
 #pragma unroll
             for (int lm = LPC / 16; lm > 0; lm >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], lm);
-            const float* sc = rec + GD_VECS * dp;
             float held[4];
 #pragma unroll
             for (int q = 0; q < 4; q++) held[q] = __shfl_sync(0xffffffffu, d[0], q * (LPC / 8), LPC);
-            {
-                const float4 a1 = *reinterpret_cast<const float4*>(sc + 16), b1 = *reinterpret_cast<const float4*>(sc + 20);
-                const float4 a2 = *reinterpret_cast<const float4*>(sc + 32), b2 = *reinterpret_cast<const float4*>(sc + 36);
-                const float4 a3 = *reinterpret_cast<const float4*>(sc + 48), b3 = *reinterpret_cast<const float4*>(sc + 52);
-                held[1] = fmaf(b1.x, held[0], fmaf(a1.x, v4.x, held[1]));
-                held[2] = fmaf(b2.x, held[0], fmaf(a2.y, v4.y, fmaf(a2.x, v4.x, held[2])));
-                held[2] = fmaf(b2.y, held[1], held[2]);
-                held[3] = fmaf(b3.x, held[0], fmaf(a3.z, v4.z, fmaf(a3.y, v4.y, fmaf(a3.x, v4.x, held[3]))));
-                held[3] = fmaf(b3.z, held[2], fmaf(b3.y, held[1], held[3]));
-            }
+            held[1] = fmaf(b1.x, held[0], fmaf(a1.x, v4.x, held[1]));
+            held[2] = fmaf(b2.x, held[0], fmaf(a2.y, v4.y, fmaf(a2.x, v4.x, held[2])));
+            held[2] = fmaf(b2.y, held[1], held[2]);
+            held[3] = fmaf(b3.x, held[0], fmaf(a3.z, v4.z, fmaf(a3.y, v4.y, fmaf(a3.x, v4.x, held[3]))));
+            held[3] = fmaf(b3.z, held[2], fmaf(b3.y, held[1], held[3]));
             // removals
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) {
-                const int i = (r4 * LPC + s) * 4;
+            for (int r4 = 0; r4 < NR / 4; r4++)
 #pragma unroll
                 for (int q = 0; q < 4; q++) {
-                    const float4 e = *reinterpret_cast<const float4*>(rec + (12 + q) * dp + i);
-                    S[4 * r4] = fmaf(-held[q], e.x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held[q], e.y, S[4 * r4 + 1]);
-                    S[4 * r4 + 2] = fmaf(-held[q], e.z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held[q], e.w, S[4 * r4 + 3]);
+                    S[4 * r4] = fmaf(-held[q], bv[q][r4].x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held[q], bv[q][r4].y, S[4 * r4 + 1]);
+                    S[4 * r4 + 2] = fmaf(-held[q], bv[q][r4].z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held[q], bv[q][r4].w, S[4 * r4 + 3]);
                 }
-            }
-            {
-                const int i = which & 3, t = b * GD_BLOCK + i;
-                const float4 c4 = *reinterpret_cast<const float4*>(sc + 16 * i + 8), e4 = *reinterpret_cast<const float4*>(sc + 16 * i + 12);
-                float o = fmaf(c4.x, v4.x, d[0]);
-                o = fmaf(c4.y, v4.y, o); o = fmaf(c4.z, v4.z, o); o = fmaf(c4.w, v4.w, o);
-                o = fmaf(e4.x, held[0], o); o = fmaf(e4.y, held[1], o); o = fmaf(e4.z, held[2], o); o = fmaf(e4.w, held[3], o);
-                if (which >= 4 && s % (LPC / 8) == 0 && col_ok && t < p.T) outp[(size_t)t * p.H * p.d] = o;
-            }
+            float o = fmaf(c4.w, v4.w, fmaf(c4.z, v4.z, fmaf(c4.y, v4.y, fmaf(c4.x, v4.x, d[0]))));
+            o = fmaf(e4.w, held[3], fmaf(e4.z, held[2], fmaf(e4.y, held[1], fmaf(e4.x, held[0], o))));
+            const int t = (st * GROUP + g) * GD_BLOCK;
+            if (stores && t + oi < p.T) outp[(size_t)t * p.H * p.d] = o;
         }
     }
     if (col_ok) {
