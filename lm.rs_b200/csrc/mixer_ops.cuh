@@ -630,11 +630,12 @@ static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const Gen
     }
 }
 
-// The scan.  Threads own state columns as in delta_scan_kernel (LPC adjacent lanes per column, NR rows each); LPC is at least 8 so
-// that the eight sums of a block can be reduced by halving: three exchange rounds leave each eighth of the lanes with one sum, the
-// rest is an ordinary reduction, and the four x_i go back to all lanes.  The lanes that hold y_i finish o_i and store it.  Records
-// arrive GD_GROUP blocks per stage through a ring of GD_RING cp.async stages.  The order of every sum is fixed.  The state is read
-// at the start (zeros when the step starts at position 0) and written back at the end.
+// The scan.  LPC adjacent lanes own CPT adjacent state columns, NR rows each in the row order of delta_scan_kernel.  What bounds it is
+// shared memory: a column needs the whole record, and only columns of the same thread share its reads, hence CPT.  LPC is at least
+// 8 CPT, so that the 8 CPT sums of a block can be reduced by halving: exchange rounds in which a lane keeps half of its sums leave
+// one sum per lane (group), the rest is an ordinary reduction, and the x_i go back to all lanes.  The lanes that hold y_i finish o_i
+// and store it.  Records arrive gd_group() blocks per stage through a ring of GD_RING cp.async stages.  The order of every sum is
+// fixed.  The state is read at the start (zeros when the step starts at position 0) and written back at the end.
 constexpr int GD_THREADS = 128, GD_RING = 4;
 struct GeneralDeltaScanParams {
     const float* rec;          // [ceil(T/4)][H][record]
@@ -645,19 +646,19 @@ struct GeneralDeltaScanParams {
     PosSrc ps;
 };
 template <int NR, int LPC> __host__ __device__ constexpr int gd_group() { return NR * LPC > 256 ? 1 : 2; }
-template <int NR, int LPC> inline size_t general_delta_scan_smem() {
-    return (size_t)GD_RING * gd_group<NR, LPC>() * (GD_VECS * NR * LPC + GD_SCALARS + GD_BLOCK * (GD_THREADS / LPC)) * 4;
+template <int NR, int LPC, int CPT> inline size_t general_delta_scan_smem() {
+    return (size_t)GD_RING * gd_group<NR, LPC>() * (GD_VECS * NR * LPC + GD_SCALARS + GD_BLOCK * (GD_THREADS / LPC * CPT)) * 4;
 }
-template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general_delta_scan_kernel(const GeneralDeltaScanParams p) {
+template <int NR, int LPC, int CPT> __global__ void __launch_bounds__(GD_THREADS) general_delta_scan_kernel(const GeneralDeltaScanParams p) {
     extern __shared__ __align__(16) float gs_sm[];
     pdl_launch();
     pdl_wait();
-    static_assert(NR % 4 == 0 && LPC >= 8 && LPC <= 32, "scan shape");
-    constexpr int cols = GD_THREADS / LPC, dp = NR * LPC, REC = GD_VECS * dp + GD_SCALARS, GROUP = gd_group<NR, LPC>();
+    static_assert(NR % 4 == 0 && LPC >= 8 * CPT && LPC <= 32, "scan shape");
+    constexpr int NS = 8 * CPT, SL = LPC / NS;   // sums of a block; lanes that end with the same one
+    constexpr int cols = GD_THREADS / LPC * CPT, dp = NR * LPC, REC = GD_VECS * dp + GD_SCALARS, GROUP = gd_group<NR, LPC>();
     constexpr int blk_fl = REC + GD_BLOCK * cols, stage_fl = GROUP * blk_fl;
     const int h = blockIdx.y;
-    const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC, j = blockIdx.x * cols + jl;
-    const bool col_ok = j < p.d;
+    const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC * CPT, j = blockIdx.x * cols + jl;
     const uint32_t pos0 = pos_of(p.ps);
     const int n_blk = (p.T + GD_BLOCK - 1) / GD_BLOCK, n_stage = (n_blk + GROUP - 1) / GROUP;
     auto stage = [&](int st) {
@@ -680,25 +681,28 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
     };
 #pragma unroll
     for (int st = 0; st < GD_RING - 1; st++) stage(st);
-    float S[NR];
+    float S[CPT][NR];
     float* sp = p.state + ((size_t)h * p.d) * p.d + j;
 #pragma unroll
-    for (int r = 0; r < NR; r++) {
-        const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
-        S[r] = (pos0 > 0 && col_ok && i < p.d) ? sp[(size_t)i * p.d] : 0.0f;
-    }
-    const int which = s / (LPC / 8);   // the sum this lane ends with: 0 .. 3 x_i, 4 .. 7 y_i
-    const int oi = which & 3;          // ... and the token of the block it finishes when it is y_i
-    const bool stores = which >= 4 && s % (LPC / 8) == 0 && col_ok;
-    float* outp = p.out + (size_t)oi * p.H * p.d + (size_t)h * p.d + j;
+    for (int cc = 0; cc < CPT; cc++)
+#pragma unroll
+        for (int r = 0; r < NR; r++) {
+            const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
+            S[cc][r] = (pos0 > 0 && j + cc < p.d && i < p.d) ? sp[(size_t)i * p.d + cc] : 0.0f;
+        }
+    const int which = s / SL;              // the sum this lane ends with: column which / 8, then 0 .. 3 x_i, 4 .. 7 y_i
+    const int oc = which >> 3, oi = which & 3;   // ... and the column and token it finishes when it is y_i
+    const bool stores = (which & 4) && s % SL == 0 && j + oc < p.d;
+    float* outp = p.out + (size_t)oi * p.H * p.d + (size_t)h * p.d + j + oc;
     // a block's dot vectors and values are read into registers while the block before it is being reduced
-    float4 nx[8][NR / 4], nv;
+    float4 nx[8][NR / 4], nv[CPT];
     auto fetch = [&](const float* rec) {
 #pragma unroll
         for (int q = 0; q < 8; q++)
 #pragma unroll
             for (int r4 = 0; r4 < NR / 4; r4++) nx[q][r4] = *reinterpret_cast<const float4*>(rec + q * dp + (r4 * LPC + s) * 4);
-        nv = *reinterpret_cast<const float4*>(rec + REC + 4 * jl);
+#pragma unroll
+        for (int cc = 0; cc < CPT; cc++) nv[cc] = *reinterpret_cast<const float4*>(rec + REC + 4 * (jl + cc));
     };
     asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
     __syncthreads();
@@ -709,7 +713,9 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
         for (int g = 0; g < GROUP; g++) {
             const float* rec = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
             const float* sc = rec + GD_VECS * dp;
-            const float4 v4 = nv;
+            float4 v4[CPT];
+#pragma unroll
+            for (int cc = 0; cc < CPT; cc++) v4[cc] = nv[cc];
             float4 kv[4][NR / 4], bv[4][NR / 4], Lv[NR / 4];
 #pragma unroll
             for (int r4 = 0; r4 < NR / 4; r4++) {
@@ -721,42 +727,48 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
             const float4 a2 = *reinterpret_cast<const float4*>(sc + 32), b2 = *reinterpret_cast<const float4*>(sc + 36);
             const float4 a3 = *reinterpret_cast<const float4*>(sc + 48), b3 = *reinterpret_cast<const float4*>(sc + 52);
             const float4 c4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 8), e4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 12);
-            float d[8];
+            float d[NS];
 #pragma unroll
-            for (int q = 0; q < 8; q++) d[q] = 0.0f;
+            for (int q = 0; q < NS; q++) d[q] = 0.0f;
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) {
+            for (int r4 = 0; r4 < NR / 4; r4++)
 #pragma unroll
-                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4], nx[q][r4].x, d[q]);
+                for (int cc = 0; cc < CPT; cc++) {
 #pragma unroll
-                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 1], nx[q][r4].y, d[q]);
+                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4], nx[q][r4].x, d[8 * cc + q]);
 #pragma unroll
-                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 2], nx[q][r4].z, d[q]);
+                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 1], nx[q][r4].y, d[8 * cc + q]);
 #pragma unroll
-                for (int q = 0; q < 8; q++) d[q] = fmaf(S[4 * r4 + 3], nx[q][r4].w, d[q]);
-            }
-            // first exchange of the reduction (eight sums over LPC lanes by halving)
+                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 2], nx[q][r4].z, d[8 * cc + q]);
+#pragma unroll
+                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 3], nx[q][r4].w, d[8 * cc + q]);
+                }
+            // one exchange of the reduction: a lane keeps m of its 2 m sums
             auto halve = [&](int m) {
-                const int lm = m * (LPC / 8);
+                const int lm = m * SL;
                 const bool up = (s & lm) != 0;
 #pragma unroll
-                for (int q = 0; q < 4; q++)
+                for (int q = 0; q < NS / 2; q++)
                     if (q < m) {
                         const float keep = up ? d[q + m] : d[q], send = up ? d[q] : d[q + m];
                         d[q] = keep + __shfl_xor_sync(0xffffffffu, send, lm);
                     }
             };
+            if (CPT > 1) halve(8);
             halve(4);
             // decay and writes: nothing here waits for the reduction
 #pragma unroll
             for (int r4 = 0; r4 < NR / 4; r4++) {
-                auto write = [&](float& x, float L, float k0, float k1, float k2, float k3) {
-                    x += fmaf(-L, x, fmaf(k3, v4.w, fmaf(k2, v4.z, fmaf(k1, v4.y, k0 * v4.x))));
-                };
-                write(S[4 * r4], Lv[r4].x, kv[0][r4].x, kv[1][r4].x, kv[2][r4].x, kv[3][r4].x);
-                write(S[4 * r4 + 1], Lv[r4].y, kv[0][r4].y, kv[1][r4].y, kv[2][r4].y, kv[3][r4].y);
-                write(S[4 * r4 + 2], Lv[r4].z, kv[0][r4].z, kv[1][r4].z, kv[2][r4].z, kv[3][r4].z);
-                write(S[4 * r4 + 3], Lv[r4].w, kv[0][r4].w, kv[1][r4].w, kv[2][r4].w, kv[3][r4].w);
+#pragma unroll
+                for (int cc = 0; cc < CPT; cc++) {
+                    auto write = [&](float& x, float L, float k0, float k1, float k2, float k3) {
+                        x += fmaf(-L, x, fmaf(k3, v4[cc].w, fmaf(k2, v4[cc].z, fmaf(k1, v4[cc].y, k0 * v4[cc].x))));
+                    };
+                    write(S[cc][4 * r4], Lv[r4].x, kv[0][r4].x, kv[1][r4].x, kv[2][r4].x, kv[3][r4].x);
+                    write(S[cc][4 * r4 + 1], Lv[r4].y, kv[0][r4].y, kv[1][r4].y, kv[2][r4].y, kv[3][r4].y);
+                    write(S[cc][4 * r4 + 2], Lv[r4].z, kv[0][r4].z, kv[1][r4].z, kv[2][r4].z, kv[3][r4].z);
+                    write(S[cc][4 * r4 + 3], Lv[r4].w, kv[0][r4].w, kv[1][r4].w, kv[2][r4].w, kv[3][r4].w);
+                }
 #pragma unroll
                 for (int q = 0; q < 4; q++) bv[q][r4] = *reinterpret_cast<const float4*>(rec + (12 + q) * dp + (r4 * LPC + s) * 4);
             }
@@ -770,36 +782,49 @@ template <int NR, int LPC> __global__ void __launch_bounds__(GD_THREADS) general
             }
             halve(1);
 #pragma unroll
-            for (int lm = LPC / 16; lm > 0; lm >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], lm);
-            float held[4];
+            for (int lm = SL / 2; lm > 0; lm >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], lm);
+            float held[CPT][4];
 #pragma unroll
-            for (int q = 0; q < 4; q++) held[q] = __shfl_sync(0xffffffffu, d[0], q * (LPC / 8), LPC);
-            held[1] = fmaf(b1.x, held[0], fmaf(a1.x, v4.x, held[1]));
-            held[2] = fmaf(b2.x, held[0], fmaf(a2.y, v4.y, fmaf(a2.x, v4.x, held[2])));
-            held[2] = fmaf(b2.y, held[1], held[2]);
-            held[3] = fmaf(b3.x, held[0], fmaf(a3.z, v4.z, fmaf(a3.y, v4.y, fmaf(a3.x, v4.x, held[3]))));
-            held[3] = fmaf(b3.z, held[2], fmaf(b3.y, held[1], held[3]));
+            for (int cc = 0; cc < CPT; cc++) {
+#pragma unroll
+                for (int q = 0; q < 4; q++) held[cc][q] = __shfl_sync(0xffffffffu, d[0], (8 * cc + q) * SL, LPC);
+            }
+            float o = d[0];
+#pragma unroll
+            for (int cc = 0; cc < CPT; cc++) {
+                float (&x)[4] = held[cc];
+                const float4 v = v4[cc];
+                x[1] = fmaf(b1.x, x[0], fmaf(a1.x, v.x, x[1]));
+                x[2] = fmaf(b2.x, x[0], fmaf(a2.y, v.y, fmaf(a2.x, v.x, x[2])));
+                x[2] = fmaf(b2.y, x[1], x[2]);
+                x[3] = fmaf(b3.x, x[0], fmaf(a3.z, v.z, fmaf(a3.y, v.y, fmaf(a3.x, v.x, x[3]))));
+                x[3] = fmaf(b3.z, x[2], fmaf(b3.y, x[1], x[3]));
+                float y = fmaf(c4.w, v.w, fmaf(c4.z, v.z, fmaf(c4.y, v.y, fmaf(c4.x, v.x, d[0]))));
+                y = fmaf(e4.w, x[3], fmaf(e4.z, x[2], fmaf(e4.y, x[1], fmaf(e4.x, x[0], y))));
+                o = oc == cc ? y : o;
+            }
             // removals
 #pragma unroll
             for (int r4 = 0; r4 < NR / 4; r4++)
 #pragma unroll
-                for (int q = 0; q < 4; q++) {
-                    S[4 * r4] = fmaf(-held[q], bv[q][r4].x, S[4 * r4]); S[4 * r4 + 1] = fmaf(-held[q], bv[q][r4].y, S[4 * r4 + 1]);
-                    S[4 * r4 + 2] = fmaf(-held[q], bv[q][r4].z, S[4 * r4 + 2]); S[4 * r4 + 3] = fmaf(-held[q], bv[q][r4].w, S[4 * r4 + 3]);
-                }
-            float o = fmaf(c4.w, v4.w, fmaf(c4.z, v4.z, fmaf(c4.y, v4.y, fmaf(c4.x, v4.x, d[0]))));
-            o = fmaf(e4.w, held[3], fmaf(e4.z, held[2], fmaf(e4.y, held[1], fmaf(e4.x, held[0], o))));
+                for (int cc = 0; cc < CPT; cc++)
+#pragma unroll
+                    for (int q = 0; q < 4; q++) {
+                        const float x = -held[cc][q];
+                        S[cc][4 * r4] = fmaf(x, bv[q][r4].x, S[cc][4 * r4]); S[cc][4 * r4 + 1] = fmaf(x, bv[q][r4].y, S[cc][4 * r4 + 1]);
+                        S[cc][4 * r4 + 2] = fmaf(x, bv[q][r4].z, S[cc][4 * r4 + 2]); S[cc][4 * r4 + 3] = fmaf(x, bv[q][r4].w, S[cc][4 * r4 + 3]);
+                    }
             const int t = (st * GROUP + g) * GD_BLOCK;
             if (stores && t + oi < p.T) outp[(size_t)t * p.H * p.d] = o;
         }
     }
-    if (col_ok) {
+#pragma unroll
+    for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
         for (int r = 0; r < NR; r++) {
             const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
-            if (i < p.d) sp[(size_t)i * p.d] = S[r];
+            if (j + cc < p.d && i < p.d) sp[(size_t)i * p.d + cc] = S[cc][r];
         }
-    }
 }
 
 // One token of the rule, one CTA per head: the projected row in, the operand-type row rms(o) * w * sigmoid(gate) out.  The low-rank
