@@ -63,9 +63,8 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
     float *proj = nullptr, *qa = nullptr, *gate = nullptr, *z = nullptr, *rec = nullptr, *fo = nullptr, *yf = nullptr, *part = nullptr, *inv = nullptr;
     AT *h = nullptr, *lat = nullptr, *att = nullptr, *act = nullptr;
     int max_proj = 0, max_ra = 0, max_q = 0, max_n = 0, max_H = 0, max_dv = 0, max_att = 0, max_ff = 0;
-    // test / measurement overrides: lanes per state column and columns per thread of the scan; one-token steps through the
-    // many-token kernels
-    int scan_lanes = 0, scan_cols = 0, step_fused = 1;
+    // test / measurement overrides: another thread layout of the scan; one-token steps through the many-token kernels
+    int scan_shape = 0, step_fused = 1;
 
     size_t n_layers() const override { return layers.size(); }
 
@@ -216,13 +215,11 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         size_t max_rec = 0;   // floats of a four-token block's records
         for (const Layer& L : layers) {
             max_heads = std::max(max_heads, L.c.H);
-            int nr, lpc, cpt;
-            scan_shape(L.c.d, &nr, &lpc, &cpt);
-            if (L.c.kind == BO_DELTA) max_rec = std::max(max_rec, (size_t)L.c.H * gd_record(nr * lpc));
+            if (L.c.kind == BO_DELTA) max_rec = std::max(max_rec, (size_t)L.c.H * gd_record(scan_rows(L.c.d)));
         }
         if (dalloc(&x, rows * width) || dalloc(&hn, rows * width) || dalloc(&d_rows, rows) || dalloc(&h, rows * width) || dalloc(&lat, rows * max_ra) ||
             dalloc(&att, rows * max_att) || dalloc(&act, rows * max_ff) || dalloc(&proj, rows * max_proj) || dalloc(&qa, rows * max_q) ||
-            dalloc(&gate, rows * max_heads) || dalloc(&z, rows * max_n) || dalloc(&rec, (rows + GD_BLOCK - 1) / GD_BLOCK * max_rec) ||
+            dalloc(&gate, rows * max_heads) || dalloc(&z, rows * max_n) || dalloc(&rec, (size_t)gd_blocks((int)rows) * max_rec) ||
             dalloc(&fo, rows * max_n) || dalloc(&yf, rows * width) || dalloc(&part, (size_t)std::max(max_H, 1) * MAX_SPLIT * (max_dv + 2)) || dalloc(&inv, rows))
             return 1;
         cap = rows;
@@ -281,27 +278,26 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         EpiParams<AT> e{}; e.out = proj; e.ldo = L.in_rows; e.scale = 1.0f;
         return this->template matmul<EPI_STORE>(st, T, h, width, L.w_in, nullptr, width, L.in_rows, e);
     }
-    // (rows per lane, lanes per column, columns per thread) of the scan for a head size
-    void scan_shape(int d, int* nr, int* lpc, int* cpt) const {
-        *cpt = scan_cols > 0 ? scan_cols : 2;
-        if (d <= 64) { *nr = 4; *lpc = 16; if (*cpt == 1 && scan_lanes == 8) { *nr = 8; *lpc = 8; } }
-        else if (d <= 128) { *nr = 8; *lpc = 16; if (scan_lanes == 32) { *nr = 4; *lpc = 32; } }
-        else if (d <= 256) { *nr = 8; *lpc = 32; }
-        else { *nr = 16; *lpc = 32; *cpt = 1; }
+    // the scan for a head size: rows per lane, lanes per column, columns and threads of a CTA follow from it
+    static int scan_rows(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : (d <= 256 ? 256 : 512)); }
+    template <int NR, int LPC, int CPT, int THREADS> int launch_scan(cudaStream_t st, const GeneralDeltaScanParams& sp) {
+        constexpr int cols = THREADS / LPC * CPT;
+        const size_t smem = general_delta_scan_smem<NR, LPC, CPT, THREADS>();
+        if (optin(general_delta_scan_kernel<NR, LPC, CPT, THREADS>, smem)) return 1;
+        return launch_k("general_delta_scan_kernel", st, pdl_now, general_delta_scan_kernel<NR, LPC, CPT, THREADS>, dim3((sp.d + cols - 1) / cols, sp.H), dim3(THREADS), smem, sp);
     }
-    template <int NR, int LPC, int CPT> int launch_scan(cudaStream_t st, const GeneralDeltaScanParams& sp) {
-        constexpr int cols = GD_THREADS / LPC * CPT;
-        const size_t smem = general_delta_scan_smem<NR, LPC, CPT>();
-        if (optin(general_delta_scan_kernel<NR, LPC, CPT>, smem)) return 1;
-        return launch_k("general_delta_scan_kernel", st, pdl_now, general_delta_scan_kernel<NR, LPC, CPT>, dim3((sp.d + cols - 1) / cols, sp.H), dim3(GD_THREADS), smem, sp);
-    }
-    int scan(cudaStream_t st, int nr, int lpc, int cpt, const GeneralDeltaScanParams& sp) {
-        if (nr == 8 && lpc == 8) return launch_scan<8, 8, 1>(st, sp);
-        if (nr == 4 && lpc == 16) return cpt == 1 ? launch_scan<4, 16, 1>(st, sp) : launch_scan<4, 16, 2>(st, sp);
-        if (nr == 8 && lpc == 16) return cpt == 1 ? launch_scan<8, 16, 1>(st, sp) : launch_scan<8, 16, 2>(st, sp);
-        if (nr == 4 && lpc == 32) return cpt == 1 ? launch_scan<4, 32, 1>(st, sp) : launch_scan<4, 32, 2>(st, sp);
-        if (nr == 8 && lpc == 32) return cpt == 1 ? launch_scan<8, 32, 1>(st, sp) : launch_scan<8, 32, 2>(st, sp);
-        return launch_scan<16, 32, 1>(st, sp);
+    int scan(cudaStream_t st, const GeneralDeltaScanParams& sp) {
+        switch (scan_rows(sp.d)) {
+            case 64:
+                if (scan_shape == 1) return launch_scan<2, 32, 2, 256>(st, sp);
+                if (scan_shape == 2) return launch_scan<4, 16, 1, 256>(st, sp);
+                return launch_scan<4, 16, 2, 128>(st, sp);
+            case 128:
+                if (scan_shape == 1) return launch_scan<4, 32, 2, 256>(st, sp);
+                return launch_scan<8, 16, 2, 128>(st, sp);
+            case 256: return launch_scan<8, 32, 2, 128>(st, sp);
+            default: return launch_scan<16, 32, 1, 128>(st, sp);
+        }
     }
     template <int RPT> int launch_step(cudaStream_t st, const GeneralDeltaStepParams<AT, WT>& p, int threads) {
         const size_t smem = ((size_t)p.ra + 5 * p.d + threads) * 4;
@@ -331,14 +327,12 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
         if (launch_k("cast_cols_kernel", st, pdl_now, cast_cols_kernel<AT>, dim3((cp.total + 255) / 256), dim3(256), 0, cp)) return 1;
         EpiParams<AT> ez{}; ez.out = z; ez.ldo = n; ez.scale = 1.0f; ez.bias = L.w0;
         if (this->template matmul<EPI_STORE>(st, T, lat, c.ra, L.w2, nullptr, c.ra, n, ez)) return 1;
-        int nr, lpc, cpt;
-        scan_shape(c.d, &nr, &lpc, &cpt);
         GeneralDeltaPreParams pp{};
-        pp.proj = proj; pp.ld = L.in_rows; pp.z = z; pp.a_bias = L.a_bias; pp.rec = rec; pp.T = T; pp.H = c.H; pp.d = c.d; pp.dp = nr * lpc; pp.decay_rate = decay_rate;
-        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3(c.H, (T + GD_BLOCK - 1) / GD_BLOCK), dim3(pp.dp), 0, pp)) return 1;
+        pp.proj = proj; pp.ld = L.in_rows; pp.z = z; pp.a_bias = L.a_bias; pp.rec = rec; pp.T = T; pp.H = c.H; pp.d = c.d; pp.dp = scan_rows(c.d); pp.decay_rate = decay_rate;
+        if (launch_k("general_delta_pre_kernel", st, pdl_now, general_delta_pre_kernel, dim3(c.H, gd_blocks(T)), dim3(pp.dp), 0, pp)) return 1;
         GeneralDeltaScanParams sp{};
-        sp.rec = rec; sp.v = proj + 2 * (size_t)n; sp.ld = L.in_rows; sp.state = L.state; sp.out = fo; sp.T = T; sp.H = c.H; sp.d = c.d; sp.ps = ps;
-        if (scan(st, nr, lpc, cpt, sp)) return 1;
+        sp.rec = rec; sp.state = L.state; sp.out = fo; sp.T = T; sp.H = c.H; sp.d = c.d; sp.ps = ps;
+        if (scan(st, sp)) return 1;
         GatedHeadNormParams<AT> gp{};
         gp.o = fo; gp.graw = proj + 3 * (size_t)n; gp.w = L.onorm; gp.w_ld = c.d; gp.eps = info.eps; gp.out = att; gp.rows = T * c.H; gp.dv = c.d; gp.H = c.H;
         gp.g_ld = L.in_rows;
@@ -399,8 +393,7 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
     }
 
     void set_model_option(const char* name, int value) override {
-        if (!strcmp(name, "scan_lanes")) { scan_lanes = value; drop_graphs(); }
-        if (!strcmp(name, "scan_cols")) { scan_cols = value; drop_graphs(); }
+        if (!strcmp(name, "scan_shape")) { scan_shape = value; drop_graphs(); }
         if (!strcmp(name, "step_fused")) { step_fused = value; drop_graphs(); }
     }
     // test access: K and V rows of an attention layer (a borrower shows its lender's)

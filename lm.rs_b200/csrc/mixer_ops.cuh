@@ -512,25 +512,29 @@ template <int NR, int LPC, int MODE = SCAN_DELTA> __global__ void __launch_bound
 // with scalars per (block, head)  A_ij = sum_c k_i k_j w_{j+1} .. w_{i-1},  B_ij the same with b_j for k_j,
 // C_ij = sum_c r_i k_j w_{j+1} .. w_i,  D_ij the same with b_j; and the state after the block is
 //     S + (sum_j (k_j w_{j+1} .. w_3) v_j^T - diag(L) S) - sum_j (b_j w_{j+1} .. w_3) held_j^T,        L = 1 - w_0 w_1 w_2 w_3.
-// Only products of decays occur, no quotients.  general_delta_pre_kernel writes the block's 17 vectors [P_i k_i (4) | P_{i+1} r_i
-// (4) | k_j w.. (4) | b_j w.. (4) | L], each padded with zeros to the scan's row count, and the scalars (token i: A_i0..3, -B_i0..3,
-// C_i0..3, -D_i0..3, zeros where the sum has no term) as one contiguous record; tokens beyond the step's end are zeros, which leave
-// the state as it is.
-constexpr int GD_BLOCK = 4, GD_VECS = 17, GD_SCALARS = 64;
-inline int gd_record(int dp) { return GD_VECS * dp + GD_SCALARS; }   // floats per (block, head), dp = padded row count
+// Only products of decays occur, no quotients.  general_delta_pre_kernel writes one contiguous record per (block, head): the block's
+// 17 vectors [P_i k_i (4) | P_{i+1} r_i (4) | k_j w.. (4) | b_j w.. (4) | L], each padded with zeros to the scan's row count; the
+// scalars [A_10 A_20 A_21 A_30 A_31 A_32 | -B the same | 4 unused | token i: C_i0..3, -D_i0..3, zeros where the sum has no term]; the
+// values [channel][token].  Tokens beyond the step's end are zeros, which leave the state as it is; whole blocks of them make the
+// number of blocks even.
+constexpr int GD_BLOCK = 4, GD_VECS = 17, GD_SCALARS = 48, GD_GROUP = 2;
+inline int gd_record(int dp) { return GD_VECS * dp + GD_SCALARS + GD_BLOCK * dp; }   // floats per (block, head), dp = padded row count
+inline int gd_blocks(int T) { return (T + GD_BLOCK * GD_GROUP - 1) / (GD_BLOCK * GD_GROUP) * GD_GROUP; }
 DN_DEVINL float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 DN_DEVINL float general_loss(float z, float rate) { return -expm1f(-rate * sigmoidf(z)); }
 struct GeneralDeltaPreParams {
     const float* proj; int ld;
     const float* z;            // [T][H*d] decay logits
     const float* a_bias;       // [H*d]
-    float* rec;                // [ceil(T/4)][H][record]
+    float* rec;                // [gd_blocks(T)][H][record]
     int T, H, d, dp;
     float decay_rate;
 };
-// where value `lane` of the reduced scalars goes in the record: A (6), B (6), C (10), D (10) as token * 16 + 4 * kind + j
-__device__ static const unsigned char gd_scalar_at[32] = {16, 32, 33, 48, 49, 50, 20, 36, 37, 52, 53, 54, 8, 24, 25, 40,
-                                                          41, 42, 56, 57, 58, 59, 12, 28, 29, 44, 45, 46, 60, 61, 62, 63};
+// where value `lane` of the reduced scalars -- A (6), B (6), C (10), D (10) -- goes in the record, and the token j of a B or D
+__device__ static const unsigned char gd_scalar_at[32] = {0, 1, 2, 3, 4, 5, 6, 7, 8, 9, 10, 11, 16, 24, 25, 32,
+                                                          33, 34, 40, 41, 42, 43, 20, 28, 29, 36, 37, 38, 44, 45, 46, 47};
+__device__ static const unsigned char gd_scalar_tok[32] = {0, 0, 0, 0, 0, 0, 0, 0, 1, 0, 1, 2, 0, 0, 0, 0,
+                                                           0, 0, 0, 0, 0, 0, 0, 0, 1, 0, 1, 2, 0, 1, 2, 3};
 // One CTA per (block, head), a thread per padded channel.  The
 // removal vectors stay unnormalised through the reductions -- B and D are linear in 1 / (sum k^2 + 1e-6) of token j.
 static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const GeneralDeltaPreParams p) {
@@ -539,8 +543,8 @@ static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const Gen
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, c = threadIdx.x;
     const int blk = blockIdx.y, h = blockIdx.x, n = p.H * p.d, t0 = blk * GD_BLOCK;
-    float* rec = p.rec + ((size_t)blk * p.H + h) * (GD_VECS * p.dp + GD_SCALARS);
-    float k[4], r[4], b[4], l[4], w[4];
+    float* rec = p.rec + ((size_t)blk * p.H + h) * (GD_VECS * p.dp + GD_SCALARS + GD_BLOCK * p.dp);
+    float k[4], r[4], b[4], l[4], w[4], v[4];
     {
         float za[4], aa[4];
         const float* q = p.proj + (size_t)t0 * p.ld + (size_t)h * p.d + c;
@@ -550,6 +554,7 @@ static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const Gen
             const bool ok = c < p.d && t0 + i < p.T;
             r[i] = ok ? q[(size_t)i * p.ld] : 0.0f;
             k[i] = ok ? q[(size_t)i * p.ld + n] : 0.0f;
+            v[i] = ok ? q[(size_t)i * p.ld + 2 * (size_t)n] : 0.0f;
             aa[i] = ok ? q[(size_t)i * p.ld + 4 * (size_t)n] : 0.0f;
             za[i] = ok ? zp[(size_t)i * n] : 0.0f;
         }
@@ -570,6 +575,7 @@ static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const Gen
 #pragma unroll
     for (int i = 1; i < GD_BLOCK; i++) L = fmaf(l[i], 1.0f - L, L);
     o[16 * p.dp] = L;
+    *reinterpret_cast<float4*>(rec + GD_VECS * p.dp + GD_SCALARS + 4 * c) = make_float4(v[0], v[1], v[2], v[3]);
     float sc[32];
     auto sums = [&](int at, int ro, const float (&u)[4]) {   // k_i . u_j for j < i, then r_i . u_j for j <= i, decayed in between
         sc[at] = k[1] * u[0];
@@ -620,89 +626,105 @@ static __global__ void __launch_bounds__(512) general_delta_pre_kernel(const Gen
     if (warp == 0) {
         float s = 0.0f;
         for (int g = 0; g < n_warps; g++) s += part[g][lane];
-        const int at = gd_scalar_at[lane];
-        if (at & 4) s *= -((at & 3) == 0 ? inv2[0] : (at & 3) == 1 ? inv2[1] : (at & 3) == 2 ? inv2[2] : inv2[3]);   // B, D: removal of token j
+        const int tok = gd_scalar_tok[lane];
+        if ((lane >= 6 && lane < 12) || lane >= 22) s *= -(tok == 0 ? inv2[0] : tok == 1 ? inv2[1] : tok == 2 ? inv2[2] : inv2[3]);
         float* so = rec + GD_VECS * p.dp;
         so[lane] = 0.0f;
-        so[lane + 32] = 0.0f;
+        if (lane < GD_SCALARS - 32) so[lane + 32] = 0.0f;
         __syncwarp();
-        so[at] = s;
+        so[gd_scalar_at[lane]] = s;
     }
 }
 
-// The scan.  LPC adjacent lanes own CPT adjacent state columns, NR rows each in the row order of delta_scan_kernel.  What bounds it is
-// shared memory: a column needs the whole record, and only columns of the same thread share its reads, hence CPT.  LPC is at least
-// 8 CPT, so that the 8 CPT sums of a block can be reduced by halving: exchange rounds in which a lane keeps half of its sums leave
-// one sum per lane (group), the rest is an ordinary reduction, and the x_i go back to all lanes.  The lanes that hold y_i finish o_i
-// and store it.  Records arrive gd_group() blocks per stage through a ring of GD_RING cp.async stages.  The order of every sum is
-// fixed.  The state is read at the start (zeros when the step starts at position 0) and written back at the end.
-constexpr int GD_THREADS = 128, GD_RING = 4;
+// The scan.  LPC adjacent lanes own CPT adjacent state columns, NR rows each: groups of V = min(NR, 4) consecutive rows, group g at
+// rows (g * LPC + s) * V.  A column needs the whole record, and only columns of the same thread share its shared-memory reads, hence
+// CPT.  LPC is at least 8 CPT, so that the 8 CPT sums of a block are reduced by halving: in every exchange a lane gives away half of
+// its sums and adds what it receives to the other half, until it holds one.  Which half it keeps is decided beforehand: lane s puts
+// the sum of vector q ^ m and of column c ^ n (m, n: bits of s) in place (c, q), so every exchange sends the upper half and keeps the
+// lower.  A lane ends with the sum of vector m in column n; lanes that end with a y_i finish o_i and store it, the x_i go back to
+// all lanes.  A block's dot vectors are read into registers while the block before it is being reduced.  Records arrive GD_GROUP
+// blocks per stage (one for the largest heads) through a ring of GD_RING cp.async stages.  The order of every sum is fixed.  The
+// state is read at the start (zeros when the step starts at position 0) and written back at the end.
+constexpr int GD_RING = 4;
 struct GeneralDeltaScanParams {
-    const float* rec;          // [ceil(T/4)][H][record]
-    const float* v; int ld;    // values of token t, head h at v + t * ld + h * d
+    const float* rec;          // [gd_blocks(T)][H][record]
     float* state;              // [H][d][d]
     float* out;                // [T][H*d]
     int T, H, d;
     PosSrc ps;
 };
-template <int NR, int LPC> __host__ __device__ constexpr int gd_group() { return NR * LPC > 256 ? 1 : 2; }
-template <int NR, int LPC, int CPT> inline size_t general_delta_scan_smem() {
-    return (size_t)GD_RING * gd_group<NR, LPC>() * (GD_VECS * NR * LPC + GD_SCALARS + GD_BLOCK * (GD_THREADS / LPC * CPT)) * 4;
+template <int NR, int LPC> __host__ __device__ constexpr int gd_group() { return NR * LPC > 256 ? 1 : GD_GROUP; }
+template <int NR, int LPC, int CPT, int THREADS> inline size_t general_delta_scan_smem() {
+    return (size_t)GD_RING * gd_group<NR, LPC>() * (GD_VECS * NR * LPC + GD_SCALARS + GD_BLOCK * (THREADS / LPC * CPT)) * 4;
 }
-template <int NR, int LPC, int CPT> __global__ void __launch_bounds__(GD_THREADS) general_delta_scan_kernel(const GeneralDeltaScanParams p) {
+template <int V> DN_DEVINL void lds_vec(const float* p, float* v) {
+    if (V == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    } else {
+        const float2 a = *reinterpret_cast<const float2*>(p);
+        v[0] = a.x; v[1] = a.y;
+    }
+}
+DN_DEVINL void cp_async16(void* smem_dst, const void* gsrc) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gsrc) : "memory");
+}
+template <int NR, int LPC, int CPT, int THREADS> __global__ void __launch_bounds__(THREADS) general_delta_scan_kernel(const GeneralDeltaScanParams p) {
     extern __shared__ __align__(16) float gs_sm[];
     pdl_launch();
     pdl_wait();
-    static_assert(NR % 4 == 0 && LPC >= 8 * CPT && LPC <= 32, "scan shape");
+    constexpr int V = NR < 4 ? NR : 4, NV = NR / V;
+    static_assert((V == 2 || V == 4) && NR % V == 0 && LPC >= 8 * CPT && LPC <= 32 && (CPT == 1 || CPT == 2), "scan shape");
     constexpr int NS = 8 * CPT, SL = LPC / NS;   // sums of a block; lanes that end with the same one
-    constexpr int cols = GD_THREADS / LPC * CPT, dp = NR * LPC, REC = GD_VECS * dp + GD_SCALARS, GROUP = gd_group<NR, LPC>();
-    constexpr int blk_fl = REC + GD_BLOCK * cols, stage_fl = GROUP * blk_fl;
+    constexpr int cols = THREADS / LPC * CPT, dp = NR * LPC, SENT = GD_VECS * dp + GD_SCALARS, REC = SENT + GD_BLOCK * dp, GROUP = gd_group<NR, LPC>();
+    constexpr int blk_fl = SENT + GD_BLOCK * cols, stage_fl = GROUP * blk_fl;   // what a CTA keeps of a record: its own columns' values
     const int h = blockIdx.y;
-    const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC * CPT, j = blockIdx.x * cols + jl;
+    const int s = threadIdx.x % LPC, jl = threadIdx.x / LPC * CPT;
+    const int which = s / SL, m = which & 7, cb = which >> 3;   // the sum this lane ends with: vector m, column cb
+    const int j0 = blockIdx.x * cols + jl;
     const uint32_t pos0 = pos_of(p.ps);
-    const int n_blk = (p.T + GD_BLOCK - 1) / GD_BLOCK, n_stage = (n_blk + GROUP - 1) / GROUP;
+    const int n_stage = (p.T + GD_BLOCK * GROUP - 1) / (GD_BLOCK * GROUP);
+    const float* src = p.rec + (size_t)h * REC;
+    const size_t step = (size_t)p.H * REC;
     auto stage = [&](int st) {
         if (st < n_stage) {
+            float* dst = gs_sm + (size_t)(st % GD_RING) * stage_fl;
+            const float* from = src + (size_t)st * GROUP * step;
 #pragma unroll
-            for (int g = 0; g < GROUP; g++) {
-                const int b = st * GROUP + g;
-                const bool real = b < n_blk;   // a block beyond the end is zeros: it leaves the state as it is
-                float* dst = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
-                const float* src = p.rec + ((size_t)(real ? b : 0) * p.H + h) * REC;
-                for (int e = threadIdx.x; e < REC / 4; e += GD_THREADS) cp_async16_zfill(dst + 4 * e, src + 4 * e, real);
-                for (int e = threadIdx.x; e < GD_BLOCK * cols; e += GD_THREADS) {
-                    const int c = e >> 2, i = e & 3, t = b * GD_BLOCK + i, jj = blockIdx.x * cols + c;   // [column][token]
-                    const bool ok = t < p.T && jj < p.d;
-                    cp_async4_zfill(dst + REC + e, ok ? p.v + (size_t)t * p.ld + (size_t)h * p.d + jj : p.v, ok);
+            for (int g = 0; g < GROUP; g++, from += step, dst += blk_fl) {
+#pragma unroll
+                for (int e0 = 0; e0 < SENT / 4; e0 += THREADS) {
+                    const int e = e0 + threadIdx.x;
+                    if (e0 + THREADS <= SENT / 4 || e < SENT / 4) cp_async16(dst + 4 * e, from + 4 * e);
                 }
+                if (threadIdx.x < cols && blockIdx.x * cols + threadIdx.x < dp)
+                    cp_async16(dst + SENT + 4 * threadIdx.x, from + SENT + 4 * (blockIdx.x * cols + threadIdx.x));
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 #pragma unroll
     for (int st = 0; st < GD_RING - 1; st++) stage(st);
-    float S[CPT][NR];
-    float* sp = p.state + ((size_t)h * p.d) * p.d + j;
+    float S[CPT][NR];   // place c holds column j0 + (c ^ cb)
+    float* sp = p.state + ((size_t)h * p.d) * p.d + j0;
 #pragma unroll
     for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
         for (int r = 0; r < NR; r++) {
-            const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
-            S[cc][r] = (pos0 > 0 && j + cc < p.d && i < p.d) ? sp[(size_t)i * p.d + cc] : 0.0f;
+            const int i = ((r / V) * LPC + s) * V + r % V, c = cc ^ cb;
+            S[cc][r] = (pos0 > 0 && j0 + c < p.d && i < p.d) ? sp[(size_t)i * p.d + c] : 0.0f;
         }
-    const int which = s / SL;              // the sum this lane ends with: column which / 8, then 0 .. 3 x_i, 4 .. 7 y_i
-    const int oc = which >> 3, oi = which & 3;   // ... and the column and token it finishes when it is y_i
-    const bool stores = (which & 4) && s % SL == 0 && j + oc < p.d;
-    float* outp = p.out + (size_t)oi * p.H * p.d + (size_t)h * p.d + j + oc;
-    // a block's dot vectors and values are read into registers while the block before it is being reduced
-    float4 nx[8][NR / 4], nv[CPT];
+    const int oi = m & 3;
+    const bool stores = (m & 4) && s % SL == 0 && j0 + cb < p.d;
+    float* outp = p.out + (size_t)oi * p.H * p.d + (size_t)h * p.d + j0 + cb;
+    float nx[8][NR], nv[CPT][4];
     auto fetch = [&](const float* rec) {
 #pragma unroll
         for (int q = 0; q < 8; q++)
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) nx[q][r4] = *reinterpret_cast<const float4*>(rec + q * dp + (r4 * LPC + s) * 4);
+            for (int r = 0; r < NV; r++) lds_vec<V>(rec + (q ^ m) * dp + (r * LPC + s) * V, nx[q] + r * V);
 #pragma unroll
-        for (int cc = 0; cc < CPT; cc++) nv[cc] = *reinterpret_cast<const float4*>(rec + REC + 4 * (jl + cc));
+        for (int cc = 0; cc < CPT; cc++) lds_vec<4>(rec + SENT + 4 * (jl + (cc ^ cb)), nv[cc]);
     };
     asm volatile("cp.async.wait_group %0;" ::"n"(GD_RING - 2) : "memory");
     __syncthreads();
@@ -713,65 +735,47 @@ template <int NR, int LPC, int CPT> __global__ void __launch_bounds__(GD_THREADS
         for (int g = 0; g < GROUP; g++) {
             const float* rec = gs_sm + (size_t)(st % GD_RING) * stage_fl + g * blk_fl;
             const float* sc = rec + GD_VECS * dp;
-            float4 v4[CPT];
+            float v[CPT][4], kv[4][NR], bv[4][NR], Lv[NR], ab[12], cd[8];
 #pragma unroll
-            for (int cc = 0; cc < CPT; cc++) v4[cc] = nv[cc];
-            float4 kv[4][NR / 4], bv[4][NR / 4], Lv[NR / 4];
+            for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) {
+                for (int q = 0; q < 4; q++) v[cc][q] = nv[cc][q];
 #pragma unroll
-                for (int q = 0; q < 4; q++) kv[q][r4] = *reinterpret_cast<const float4*>(rec + (8 + q) * dp + (r4 * LPC + s) * 4);
-                Lv[r4] = *reinterpret_cast<const float4*>(rec + 16 * dp + (r4 * LPC + s) * 4);
+            for (int r = 0; r < NV; r++) {
+#pragma unroll
+                for (int q = 0; q < 4; q++) lds_vec<V>(rec + (8 + q) * dp + (r * LPC + s) * V, kv[q] + r * V);
+                lds_vec<V>(rec + 16 * dp + (r * LPC + s) * V, Lv + r * V);
             }
-            const float4 a1 = *reinterpret_cast<const float4*>(sc + 16), b1 = *reinterpret_cast<const float4*>(sc + 20);
-            const float4 a2 = *reinterpret_cast<const float4*>(sc + 32), b2 = *reinterpret_cast<const float4*>(sc + 36);
-            const float4 a3 = *reinterpret_cast<const float4*>(sc + 48), b3 = *reinterpret_cast<const float4*>(sc + 52);
-            const float4 c4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 8), e4 = *reinterpret_cast<const float4*>(sc + 16 * oi + 12);
+#pragma unroll
+            for (int q = 0; q < 3; q++) lds_vec<4>(sc + 4 * q, ab + 4 * q);
+            lds_vec<4>(sc + 16 + 8 * oi, cd);
+            lds_vec<4>(sc + 20 + 8 * oi, cd + 4);
             float d[NS];
 #pragma unroll
             for (int q = 0; q < NS; q++) d[q] = 0.0f;
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++)
+            for (int r = 0; r < NR; r++)
 #pragma unroll
-                for (int cc = 0; cc < CPT; cc++) {
+                for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
-                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4], nx[q][r4].x, d[8 * cc + q]);
-#pragma unroll
-                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 1], nx[q][r4].y, d[8 * cc + q]);
-#pragma unroll
-                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 2], nx[q][r4].z, d[8 * cc + q]);
-#pragma unroll
-                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][4 * r4 + 3], nx[q][r4].w, d[8 * cc + q]);
-                }
-            // one exchange of the reduction: a lane keeps m of its 2 m sums
-            auto halve = [&](int m) {
-                const int lm = m * SL;
-                const bool up = (s & lm) != 0;
+                    for (int q = 0; q < 8; q++) d[8 * cc + q] = fmaf(S[cc][r], nx[q][r], d[8 * cc + q]);
+            auto halve = [&](int k) {   // 2 k sums -> k
 #pragma unroll
                 for (int q = 0; q < NS / 2; q++)
-                    if (q < m) {
-                        const float keep = up ? d[q + m] : d[q], send = up ? d[q] : d[q + m];
-                        d[q] = keep + __shfl_xor_sync(0xffffffffu, send, lm);
-                    }
+                    if (q < k) d[q] += __shfl_xor_sync(0xffffffffu, d[q + k], k * SL);
             };
             if (CPT > 1) halve(8);
             halve(4);
             // decay and writes: nothing here waits for the reduction
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++) {
+            for (int r = 0; r < NR; r++)
 #pragma unroll
-                for (int cc = 0; cc < CPT; cc++) {
-                    auto write = [&](float& x, float L, float k0, float k1, float k2, float k3) {
-                        x += fmaf(-L, x, fmaf(k3, v4[cc].w, fmaf(k2, v4[cc].z, fmaf(k1, v4[cc].y, k0 * v4[cc].x))));
-                    };
-                    write(S[cc][4 * r4], Lv[r4].x, kv[0][r4].x, kv[1][r4].x, kv[2][r4].x, kv[3][r4].x);
-                    write(S[cc][4 * r4 + 1], Lv[r4].y, kv[0][r4].y, kv[1][r4].y, kv[2][r4].y, kv[3][r4].y);
-                    write(S[cc][4 * r4 + 2], Lv[r4].z, kv[0][r4].z, kv[1][r4].z, kv[2][r4].z, kv[3][r4].z);
-                    write(S[cc][4 * r4 + 3], Lv[r4].w, kv[0][r4].w, kv[1][r4].w, kv[2][r4].w, kv[3][r4].w);
-                }
+                for (int cc = 0; cc < CPT; cc++)
+                    S[cc][r] += fmaf(-Lv[r], S[cc][r], fmaf(kv[3][r], v[cc][3], fmaf(kv[2][r], v[cc][2], fmaf(kv[1][r], v[cc][1], kv[0][r] * v[cc][0]))));
 #pragma unroll
-                for (int q = 0; q < 4; q++) bv[q][r4] = *reinterpret_cast<const float4*>(rec + (12 + q) * dp + (r4 * LPC + s) * 4);
-            }
+            for (int r = 0; r < NV; r++)
+#pragma unroll
+                for (int q = 0; q < 4; q++) lds_vec<V>(rec + (12 + q) * dp + (r * LPC + s) * V, bv[q] + r * V);
             halve(2);
             if (g + 1 < GROUP) {
                 fetch(rec + blk_fl);
@@ -785,35 +789,31 @@ template <int NR, int LPC, int CPT> __global__ void __launch_bounds__(GD_THREADS
             for (int lm = SL / 2; lm > 0; lm >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], lm);
             float held[CPT][4];
 #pragma unroll
-            for (int cc = 0; cc < CPT; cc++) {
+            for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
-                for (int q = 0; q < 4; q++) held[cc][q] = __shfl_sync(0xffffffffu, d[0], (8 * cc + q) * SL, LPC);
-            }
-            float o = d[0];
+                for (int q = 0; q < 4; q++) held[cc][q] = __shfl_sync(0xffffffffu, d[0], (8 * (cc ^ cb) + q) * SL, LPC);
 #pragma unroll
             for (int cc = 0; cc < CPT; cc++) {
                 float (&x)[4] = held[cc];
-                const float4 v = v4[cc];
-                x[1] = fmaf(b1.x, x[0], fmaf(a1.x, v.x, x[1]));
-                x[2] = fmaf(b2.x, x[0], fmaf(a2.y, v.y, fmaf(a2.x, v.x, x[2])));
-                x[2] = fmaf(b2.y, x[1], x[2]);
-                x[3] = fmaf(b3.x, x[0], fmaf(a3.z, v.z, fmaf(a3.y, v.y, fmaf(a3.x, v.x, x[3]))));
-                x[3] = fmaf(b3.z, x[2], fmaf(b3.y, x[1], x[3]));
-                float y = fmaf(c4.w, v.w, fmaf(c4.z, v.z, fmaf(c4.y, v.y, fmaf(c4.x, v.x, d[0]))));
-                y = fmaf(e4.w, x[3], fmaf(e4.z, x[2], fmaf(e4.y, x[1], fmaf(e4.x, x[0], y))));
-                o = oc == cc ? y : o;
+                const float (&u)[4] = v[cc];
+                x[1] = fmaf(ab[6], x[0], fmaf(ab[0], u[0], x[1]));
+                x[2] = fmaf(ab[7], x[0], fmaf(ab[2], u[1], fmaf(ab[1], u[0], x[2])));
+                x[2] = fmaf(ab[8], x[1], x[2]);
+                x[3] = fmaf(ab[9], x[0], fmaf(ab[5], u[2], fmaf(ab[4], u[1], fmaf(ab[3], u[0], x[3]))));
+                x[3] = fmaf(ab[11], x[2], fmaf(ab[10], x[1], x[3]));
             }
             // removals
 #pragma unroll
-            for (int r4 = 0; r4 < NR / 4; r4++)
+            for (int q = 0; q < 4; q++)
 #pragma unroll
                 for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
-                    for (int q = 0; q < 4; q++) {
-                        const float x = -held[cc][q];
-                        S[cc][4 * r4] = fmaf(x, bv[q][r4].x, S[cc][4 * r4]); S[cc][4 * r4 + 1] = fmaf(x, bv[q][r4].y, S[cc][4 * r4 + 1]);
-                        S[cc][4 * r4 + 2] = fmaf(x, bv[q][r4].z, S[cc][4 * r4 + 2]); S[cc][4 * r4 + 3] = fmaf(x, bv[q][r4].w, S[cc][4 * r4 + 3]);
-                    }
+                    for (int r = 0; r < NR; r++) S[cc][r] = fmaf(-held[cc][q], bv[q][r], S[cc][r]);
+            float o = d[0];   // y_i of place 0's column, when this lane holds one
+#pragma unroll
+            for (int q = 0; q < 4; q++) o = fmaf(cd[q], v[0][q], o);
+#pragma unroll
+            for (int q = 0; q < 4; q++) o = fmaf(cd[4 + q], held[0][q], o);
             const int t = (st * GROUP + g) * GD_BLOCK;
             if (stores && t + oi < p.T) outp[(size_t)t * p.H * p.d] = o;
         }
@@ -822,8 +822,8 @@ template <int NR, int LPC, int CPT> __global__ void __launch_bounds__(GD_THREADS
     for (int cc = 0; cc < CPT; cc++)
 #pragma unroll
         for (int r = 0; r < NR; r++) {
-            const int i = ((r >> 2) * LPC + s) * 4 + (r & 3);
-            if (j + cc < p.d && i < p.d) sp[(size_t)i * p.d + cc] = S[cc][r];
+            const int i = ((r / V) * LPC + s) * V + r % V, c = cc ^ cb;
+            if (j0 + c < p.d && i < p.d) sp[(size_t)i * p.d + c] = S[cc][r];
         }
 }
 
