@@ -57,7 +57,6 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
     float* final_norm = nullptr;
     float softcap = 0.0f, decay_rate = (float)exp(-0.5);
     float* shift_rows = nullptr;   // [2][layers][width]
-    unsigned int* counter = nullptr;
     uint32_t next_pos = 0;         // where the recurrent states and shift rows stand
     // scratch for `cap` rows
     float *proj = nullptr, *qa = nullptr, *gate = nullptr, *z = nullptr, *rec = nullptr, *fo = nullptr, *yf = nullptr, *part = nullptr, *inv = nullptr;
@@ -171,9 +170,8 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
             return 1;
         layers.resize(jl.arr.size());
         const size_t nl = layers.size();
-        if (dalloc(&shift_rows, 2 * nl * width) || dalloc(&counter, 1)) return 1;
+        if (dalloc(&shift_rows, 2 * nl * width)) return 1;
         GCK(cudaMemset(shift_rows, 0, 2 * nl * width * 4));
-        GCK(cudaMemset(counter, 0, 4));
         for (size_t li = 0; li < nl; li++) {
             Layer& L = layers[li];
             if (parse_layer(jl.arr[li], li, L.c)) return 1;
@@ -251,7 +249,11 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
             p.w_next = nx.w; p.h = h; p.ldh = width;
             if (nx.shift) { p.mu = nx.shift->mu; p.prev = nx.shift->prev; }
         }
-        if (launch_k("resnorm_rows_kernel", st, pdl_now, resnorm_rows_kernel<AT>, dim3(T), dim3(256), 0, p)) return 1;
+        if (T == 1) {
+            const int threads = std::min(1024, (width + 31) / 32 * 32);
+            return launch_k("resnorm_rows_kernel", st, pdl_now, resnorm_rows_kernel<AT, true>, dim3(1), dim3(threads), 0, p);
+        }
+        if (launch_k("resnorm_rows_kernel", st, pdl_now, resnorm_rows_kernel<AT, false>, dim3(T), dim3(256), 0, p)) return 1;
         if (!two) return 0;
         NormShiftRowsParams<AT> sp{};
         sp.x = x; sp.ldx = width; sp.inv = inv; sp.w = nx.w; sp.mu = nx.shift->mu; sp.prev_in = nx.shift->prev; sp.prev_out = nx.shift->prev + layers.size() * width;
@@ -262,13 +264,6 @@ template <typename AT, typename WT> class BolapelModel : public DenseModel<AT, W
     // a sublayer's last product a . w^T, its norm, the residual and the next sublayer's input
     int sublayer_out(cudaStream_t st, int T, const AT* a, int K, const WT* w, const float* wb, const Next& nx, const PosSrc& ps) {
         EpiParams<AT> e{}; e.out = yf; e.ldo = width; e.scale = 1.0f;
-        if (T == 1) {   // one row: the CTA that finishes last goes on with the norms
-            GemvRowsParams<AT, WT> p{};
-            p.a = a; p.w = w; p.K = K; p.O = width; p.e = e;
-            p.ln.counter = counter; p.ln.w = wb; p.ln.eps = info.eps; p.ln.x = x; p.ln.h = h; p.ln.w_next = nx.w; p.ln.ps = ps;
-            if (nx.shift) { p.ln.mu = nx.shift->mu; p.ln.prev = nx.shift->prev; }
-            return this->template launch_gemv<EPI_STORE, NORM_NONE, TAIL_RMS>(st, p);
-        }
         if (this->template matmul<EPI_STORE>(st, T, a, K, w, nullptr, K, width, e)) return 1;
         return residual_rows(st, T, wb, nx, ps);
     }

@@ -289,9 +289,9 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         gemm_tiled_kernel<AT, WT, EPI><<<dim3((O + 63) / 64, (std::min(T, max_group_rows) + 63) / 64, n_groups), 256, 0, st>>>(p);
         return check_launch("gemm_tiled_kernel");
     }
-    template <int EPI, int NORM, int TAIL = TAIL_LAYER> int launch_gemv(cudaStream_t st, GemvRowsParams<AT, WT> p, int nb = 1) {
+    template <int EPI, int NORM> int launch_gemv(cudaStream_t st, GemvRowsParams<AT, WT> p, int nb = 1) {
         const size_t smem = ((size_t)((p.K + 3) & ~3) + 36 + 2 * 8 + 4) * 4;
-        if (optin(gemv_rows_kernel<AT, WT, EPI, NORM, TAIL>, smem)) return 1;
+        if (optin(gemv_rows_kernel<AT, WT, EPI, NORM>, smem)) return 1;
         const int rows_per_cta = EPI == EPI_GLU ? 8 : 16;
         int grid = (p.O + rows_per_cta - 1) / rows_per_cta;
         // few rows: the warps of a CTA split K instead (two row pairs per CTA)
@@ -299,7 +299,7 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         if (p.ksplit) grid = (p.O + 3) / 4;
         p.pdl = pdl_now ? 1 : 0;
         grid = std::max(1, std::min(grid, sms * 4));
-        return launch_k("gemv_rows_kernel", st, pdl_now, gemv_rows_kernel<AT, WT, EPI, NORM, TAIL>, dim3(grid, nb), dim3(256), smem, p);
+        return launch_k("gemv_rows_kernel", st, pdl_now, gemv_rows_kernel<AT, WT, EPI, NORM>, dim3(grid, nb), dim3(256), smem, p);
     }
 
     template <int RW, int NI, bool SIG> int launch_attn_t(cudaStream_t st, AttnRowsParams<AT> p, int grid_x, int grid_y) {

@@ -238,45 +238,52 @@ template <typename AT> __global__ void __launch_bounds__(256) layernorm_rows_ker
 }
 
 // ---- normed sublayer outputs into one residual stream, with the next norm behind -------------------------------------------
-// One row through a whole CTA: load(c) gives the sublayer's output; with wb
-//     x[c] <- x[c] + load(c) / sqrt(mean(load^2) + eps) * wb[c]
+// One row through a whole CTA: y is the sublayer's output; with wb
+//     x[c] <- x[c] + y[c] / sqrt(mean(y^2) + eps) * wb[c]
 // (without wb the row is x itself), then with w_next the next sublayer's input
 //     g[c] = x[c] / sqrt(mean(x^2) + eps) * w_next[c];      h[c] = g[c] + (before[c] - g[c]) * mu[c]        (mu: token shift)
 // where `before` is the previous token's g: read from prev (zeros when `fresh`, the first token of a sequence), which then takes
-// this token's g.  inv_out asks for the factor 1 / sqrt(mean(x^2) + eps) instead of h.  Rows up to SANDWICH_CACHE * blockDim.x
-// columns stay in registers; longer ones are loaded again.
-constexpr int SANDWICH_CACHE = 12;
-template <typename AT, typename F>
-DN_DEVINL void sandwich_row(F load, int n, float* x, const float* wb, float eps, float* red, const float* w_next, const float* mu, float* prev,
+// this token's g.  inv_out asks for the factor 1 / sqrt(mean(x^2) + eps) instead of h.  Rows up to CACHE * blockDim.x columns stay
+// in registers; longer ones are loaded again.  EARLY: the weights are loaded with the row instead of when they are needed (a single
+// row is nothing but latency).
+template <typename AT, int CACHE, bool EARLY>
+DN_DEVINL void sandwich_row(const float* y, int n, float* x, const float* wb, float eps, float* red, const float* w_next, const float* mu, float* prev,
                             bool fresh, AT* h, float* inv_out) {
-    const bool cached = n <= SANDWICH_CACHE * (int)blockDim.x;
-    float v[SANDWICH_CACHE];
+    const bool cached = n <= CACHE * (int)blockDim.x;
+    float v[CACHE];
+    float wv[EARLY ? CACHE : 1], mv[EARLY ? CACHE : 1], pv[EARLY ? CACHE : 1];
     float ss = 0.0f;
     if (cached) {
-        float xv[SANDWICH_CACHE];
+        float xv[CACHE], bv[EARLY ? CACHE : 1];
 #pragma unroll
-        for (int i = 0; i < SANDWICH_CACHE; i++) {
+        for (int i = 0; i < CACHE; i++) {
             const int c = threadIdx.x + i * blockDim.x;
-            v[i] = c < n ? (wb ? load(c) : x[c]) : 0.0f;
+            v[i] = c < n ? (wb ? y[c] : x[c]) : 0.0f;
             xv[i] = c < n && wb ? x[c] : 0.0f;
+            if (EARLY) {
+                bv[i] = c < n && wb ? wb[c] : 0.0f;
+                wv[i] = c < n && w_next ? w_next[c] : 0.0f;
+                mv[i] = c < n && mu ? mu[c] : 0.0f;
+                pv[i] = c < n && mu && !fresh ? prev[c] : 0.0f;
+            }
         }
 #pragma unroll
-        for (int i = 0; i < SANDWICH_CACHE; i++) ss = fmaf(v[i], v[i], ss);
+        for (int i = 0; i < CACHE; i++) ss = fmaf(v[i], v[i], ss);
         if (wb) {
             const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
             ss = 0.0f;
 #pragma unroll
-            for (int i = 0; i < SANDWICH_CACHE; i++) {
+            for (int i = 0; i < CACHE; i++) {
                 const int c = threadIdx.x + i * blockDim.x;
-                if (c < n) { v[i] = xv[i] + v[i] * inv * wb[c]; x[c] = v[i]; }
+                if (c < n) { v[i] = xv[i] + v[i] * inv * (EARLY ? bv[i] : wb[c]); x[c] = v[i]; }
                 ss = fmaf(v[i], v[i], ss);
             }
         }
     } else if (wb) {
-        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = load(c); ss = fmaf(a, a, ss); }
+        for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(y[c], y[c], ss);
         const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
         ss = 0.0f;
-        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = x[c] + load(c) * inv * wb[c]; x[c] = a; ss = fmaf(a, a, ss); }
+        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = x[c] + y[c] * inv * wb[c]; x[c] = a; ss = fmaf(a, a, ss); }
     } else {
         for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
     }
@@ -286,23 +293,25 @@ DN_DEVINL void sandwich_row(F load, int n, float* x, const float* wb, float eps,
         if (threadIdx.x == 0) *inv_out = inv;
         return;
     }
-    auto finish = [&](int c, float a) {
-        a = a * inv * w_next[c];
+    auto finish = [&](int c, float a, float w, float before, float m) {
+        a = a * inv * w;
         if (mu) {
-            const float before = fresh ? 0.0f : prev[c];
             prev[c] = a;
-            a = a + (before - a) * mu[c];
+            a = a + (before - a) * m;
         }
         from_f(h[c], a);
     };
     if (cached) {
 #pragma unroll
-        for (int i = 0; i < SANDWICH_CACHE; i++) {
+        for (int i = 0; i < CACHE; i++) {
             const int c = threadIdx.x + i * blockDim.x;
-            if (c < n) finish(c, v[i]);
+            if (c >= n) continue;
+            if (EARLY) finish(c, v[i], wv[i], pv[i], mv[i]);
+            else finish(c, v[i], w_next[c], mu && !fresh ? prev[c] : 0.0f, mu ? mu[c] : 0.0f);
         }
     } else {
-        for (int c = threadIdx.x; c < n; c += blockDim.x) finish(c, x[c]);   // this thread stored it above
+        for (int c = threadIdx.x; c < n; c += blockDim.x)   // this thread stored x[c] above
+            finish(c, x[c], w_next[c], mu && !fresh ? prev[c] : 0.0f, mu ? mu[c] : 0.0f);
     }
 }
 template <typename AT> struct ResNormRowsParams {
@@ -313,14 +322,14 @@ template <typename AT> struct ResNormRowsParams {
     float* inv_out;                                // [T]: many rows: the factors for norm_shift_rows_kernel
     PosSrc ps;
 };
-template <typename AT> __global__ void __launch_bounds__(256) resnorm_rows_kernel(const ResNormRowsParams<AT> p) {
+// ONE: a step of one row (up to 1024 threads); otherwise 256 threads per row
+template <typename AT, bool ONE> __global__ void __launch_bounds__(ONE ? 1024 : 256) resnorm_rows_kernel(const ResNormRowsParams<AT> p) {
     __shared__ float red[33];
     pdl_launch();
     pdl_wait();
     const int r = blockIdx.x;
-    const float* y = p.wb ? p.y + (size_t)r * p.ldy : nullptr;
-    sandwich_row<AT>([&](int c) { return y[c]; }, p.n, p.x + (size_t)r * p.ldx, p.wb, p.eps, red, p.w_next, p.mu, p.prev, p.mu && pos_of(p.ps) == 0,
-                     p.h ? p.h + (size_t)r * p.ldh : nullptr, p.inv_out ? p.inv_out + r : nullptr);
+    sandwich_row<AT, ONE ? 4 : 12, ONE>(p.wb ? p.y + (size_t)r * p.ldy : nullptr, p.n, p.x + (size_t)r * p.ldx, p.wb, p.eps, red, p.w_next, p.mu, p.prev,
+                                        p.mu && pos_of(p.ps) == 0, p.h ? p.h + (size_t)r * p.ldh : nullptr, p.inv_out ? p.inv_out + r : nullptr);
 }
 // g_t = x_t * inv[t] * w;  h_t = g_t + (g_{t-1} - g_t) * mu.  Row -1 is prev_in (zeros for a step at position 0); the last row's g
 // goes to prev_out (another buffer: blocks of the grid still read prev_in).  A thread walks NORM_SHIFT_ROWS rows of one column.
@@ -533,14 +542,10 @@ enum { NORM_NONE = 0, NORM_RMS = 1, NORM_TANH = 2, NORM_LAYER = 3 };
 // -- every CTA takes a ticket from *counter after its stores -- sends the row e.out[0 .. O) through a layer norm into the
 // residual stream, x <- x + ls * LN(row) w, and writes x again in the operand type to h.  Nobody waits for anybody: the last
 // ticket simply falls to whoever comes last, and that CTA puts the counter back to zero.
-// The RMS form (kernels instantiated with TAIL_RMS) sends the row through sandwich_row instead: x <- x + rms(row) w, and the next
-// sublayer's input rms(x) w_next, token-shifted when mu is given, to h.
-enum { TAIL_LAYER = 0, TAIL_RMS = 1 };
 template <typename AT> struct LnTail {
     unsigned int* counter;
     const float* w; const float* ls; float eps;
     float* x; AT* h;
-    const float* w_next; const float* mu; float* prev; PosSrc ps;   // RMS form
 };
 template <typename AT, typename WT> struct GemvRowsParams {
     const AT* a;              // [K] input row (NORM_NONE)
@@ -620,7 +625,7 @@ DN_DEVINL void dot_rows(const WT* const (&w)[NR], const float* __restrict__ xs, 
 #pragma unroll
     for (int r = 0; r < NR; r++) out[r] = warp_sum(acc[r]);
 }
-template <typename AT, typename WT, int EPI, int NORM, int TAIL = TAIL_LAYER>
+template <typename AT, typename WT, int EPI, int NORM>
 static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsParams<AT, WT> pp) {
     extern __shared__ __align__(16) float gv_xs[];   // [K rounded up to 4] the input row as f32, then reduction slots
     GemvRowsParams<AT, WT> p = pp;
@@ -727,11 +732,7 @@ static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsPar
         if (last) {
             __threadfence();
             const float* row = p.e.out;
-            if (TAIL == TAIL_RMS)
-                sandwich_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.x, p.ln.w, p.ln.eps, red, p.ln.w_next, p.ln.mu, p.ln.prev,
-                                 p.ln.mu && pos_of(p.ln.ps) == 0, p.ln.h, nullptr);
-            else
-                layernorm_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.w, p.ln.eps, red, p.ln.x, p.ln.ls, nullptr, p.ln.h);
+            layernorm_row<AT>([&](int c) { return __ldcg(row + c); }, p.O, p.ln.w, p.ln.eps, red, p.ln.x, p.ln.ls, nullptr, p.ln.h);
             if (threadIdx.x == 0) *p.ln.counter = 0u;
         }
     }
