@@ -977,6 +977,27 @@ template <typename AT> __global__ void __launch_bounds__(128) gated_headnorm_ker
     AT* dst = p.out_ld > 0 ? p.out + (size_t)t * p.out_ld + (size_t)hh * p.dv : p.out + (size_t)r * p.dv;
     const float* w = p.w + (size_t)hh * p.w_ld;
     float ss = 0.0f;
+    constexpr int HN_CACHE = 4;   // heads up to 32 * HN_CACHE: everything is loaded before the reduction
+    if (p.dv <= 32 * HN_CACHE) {
+        float ov[HN_CACHE], gv[HN_CACHE], wv[HN_CACHE];
+#pragma unroll
+        for (int i = 0; i < HN_CACHE; i++) {
+            const int c = lane + 32 * i;
+            ov[i] = c < p.dv ? o[c] : 0.0f;
+            gv[i] = c < p.dv ? gr[c] : 0.0f;
+            wv[i] = c < p.dv ? w[c] : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < HN_CACHE; i++) ss += ov[i] * ov[i];
+        const float inv = (p.has_out_scale ? p.out_scale : 1.0f) / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
+#pragma unroll
+        for (int i = 0; i < HN_CACHE; i++) {
+            const int c = lane + 32 * i;
+            const float sg = 1.0f / (1.0f + expf(-gv[i]));
+            if (c < p.dv) from_f(dst[c], ov[i] * inv * wv[i] * (p.gate_silu ? gv[i] * sg : sg));
+        }
+        return;
+    }
     for (int c = lane; c < p.dv; c += 32) ss += o[c] * o[c];
     ss = warp_sum(ss);
     const float inv = (p.has_out_scale ? p.out_scale : 1.0f) / sqrtf(ss / (float)p.dv + p.eps);
