@@ -202,7 +202,6 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_const
                 for (int j = 0; j < 32; j++) {
                     float val = __uint_as_float(v[j]);
                     if constexpr (GLU) val = glu_apply(p.e, val, __uint_as_float(u[j]));
-                    if constexpr (EPI == EPI_ACT) val = act_apply(p.e, val);
                     stg[lane * 33 + j] = val;
                 }
                 __syncwarp();
@@ -237,9 +236,14 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_const
                         }
                     } else {
                         __nv_bfloat16* __restrict__ dst = p.e.act + (size_t)t0 * p.e.lda + o;
+                        const float bias = EPI == EPI_ACT && p.e.bias ? p.e.bias[o] : 0.0f;
 #pragma unroll 8
                         for (int r = 0; r < 32; r++)
-                            if (t0 + r < row_end) dst[(size_t)r * p.e.lda] = __float2bfloat16_rn(stg[r * 33 + lane]);
+                            if (t0 + r < row_end) {
+                                float a = stg[r * 33 + lane];
+                                if constexpr (EPI == EPI_ACT) a = act_apply(p.e, a + bias);
+                                dst[(size_t)r * p.e.lda] = __float2bfloat16_rn(a);
+                            }
                     }
                 }
                 __syncwarp();

@@ -162,13 +162,44 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         return 0;
     }
 
+    int upload_host(const std::vector<float>& v, WT* dst) {   // host floats in the operand type
+        if (std::is_same<WT, float>::value) { GCK(cudaMemcpy(dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice)); return 0; }
+        std::vector<__nv_bfloat16> tmp(v.size());
+        for (size_t i = 0; i < v.size(); i++) tmp[i] = __float2bfloat16_rn(v[i]);
+        GCK(cudaMemcpy(dst, tmp.data(), tmp.size() * 2, cudaMemcpyHostToDevice));
+        return 0;
+    }
+
     int load_vec(const SafeTensors& st, const std::string& name, int n, float** out) {
         const StTensor* t = nullptr;
         return need(st, name, {n}, &t) || upload_f32(t, out);
     }
+    // a norm weight stored around zero: 1 + w
+    int load_offset_vec(const SafeTensors& st, const std::string& name, int n, float** out) {
+        const StTensor* t = nullptr;
+        if (need(st, name, {n}, &t)) return 1;
+        std::vector<float> v((size_t)n);
+        for (int i = 0; i < n; i++) v[i] = 1.0f + (t->dtype == "BF16" ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(t->data)[i]) : reinterpret_cast<const float*>(t->data)[i]);
+        if (dalloc(out, v.size())) return 1;
+        GCK(cudaMemcpy(*out, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+        return 0;
+    }
     int load_mat_f32(const SafeTensors& st, const std::string& name, int rows, int cols, float** out) {
         const StTensor* t = nullptr;
         return need(st, name, {rows, cols}, &t) || upload_f32(t, out);
+    }
+    // the same for several matrices stacked into one
+    int load_stack_f32(const SafeTensors& st, const std::vector<std::pair<std::string, int>>& parts, int K, float** out) {
+        std::vector<float> host;
+        for (const auto& pr : parts) {
+            const StTensor* t = nullptr;
+            if (need(st, pr.first, {pr.second, K}, &t)) return 1;
+            for (size_t i = 0; i < t->numel(); i++)
+                host.push_back(t->dtype == "BF16" ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(t->data)[i]) : reinterpret_cast<const float*>(t->data)[i]);
+        }
+        if (dalloc(out, host.size())) return 1;
+        GCK(cudaMemcpy(*out, host.data(), host.size() * 4, cudaMemcpyHostToDevice));
+        return 0;
     }
     // matrices stacked into one: rows of `parts` in order, then zero rows up to a multiple of `row_multiple`
     int load_stack(const SafeTensors& st, const std::vector<std::pair<std::string, int>>& parts, int K, WT** out, int* rows_out, int row_multiple = 1) {
@@ -290,13 +321,14 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         return check_launch("gemm_tiled_kernel");
     }
     template <int EPI, int NORM> int launch_gemv(cudaStream_t st, GemvRowsParams<AT, WT> p, int nb = 1) {
-        const size_t smem = ((size_t)((p.K + 3) & ~3) + 36 + 2 * 8 + 4) * 4;
+        const int K = std::max(p.K, p.extra.w ? p.extra.K : 0), O = std::max(p.O, p.extra.w ? p.extra.O : 0);
+        const size_t smem = ((size_t)((K + 3) & ~3) + 36 + 2 * 8 + 4) * 4;
         if (optin(gemv_rows_kernel<AT, WT, EPI, NORM>, smem)) return 1;
         const int rows_per_cta = EPI == EPI_GLU ? 8 : 16;
-        int grid = (p.O + rows_per_cta - 1) / rows_per_cta;
+        int grid = (O + rows_per_cta - 1) / rows_per_cta;
         // few rows: the warps of a CTA split K instead (two row pairs per CTA)
         p.ksplit = EPI != EPI_GLU && grid < 2 * sms && p.K % Vec16<WT>::N == 0 && p.K >= 1024;
-        if (p.ksplit) grid = (p.O + 3) / 4;
+        if (p.ksplit) grid = (O + 3) / 4;
         p.pdl = pdl_now ? 1 : 0;
         grid = std::max(1, std::min(grid, sms * 4));
         return launch_k("gemv_rows_kernel", st, pdl_now, gemv_rows_kernel<AT, WT, EPI, NORM>, dim3(grid, nb), dim3(256), smem, p);

@@ -1,13 +1,14 @@
 // dense_ops.cuh -- kernels for models with unquantized weights (bf16 or f32 operands, f32 accumulation): the building
 // blocks a folder-based architecture (arch.h) composes.  Every constant of a mechanism is a parameter, so that another
 // architecture can use the same kernel:
-//   embed_rows_kernel        token embedding + optional hashed bigram embedding of (previous token, token)
+//   embed_rows_kernel        token embedding + optional hashed bigram embedding of (previous token, token), optionally scaled
 //   rmsnorm_rows_kernel      x / sqrt(mean(x^2) + eps) * w per row, optional row gather, output in the operand type
 //   tanhnorm_rows_kernel     tanh(alpha * x) * w + b per element (a norm without statistics), same gather and output
 //   layernorm_rows_kernel    (x - mean) / sqrt(var + eps) * w per row; the result is stored, or scaled per column and added
 //                            to the residual stream, and the row that comes out is also written in the operand type
 //   resnorm_rows_kernel      residual <- residual + rms(sublayer output) * w, then the next sublayer's RMS norm of it (or that
-//                            row's factor alone), optionally mixed with the previous token's normed row (token shift)
+//                            row's factor alone, or the residual row as it is in the operand type), optionally mixed with the
+//                            previous token's normed row (token shift)
 //   norm_shift_rows_kernel   the token shift of many rows whose norm factors are known
 //   gemv_rows_kernel         one token row:  weights streamed once (HBM-bound), optional fused RMS-norm prologue,
 //                            epilogues: store*scale+bias | x += ls * f(acc) + lb | act(gate) * up | store in the operand
@@ -84,8 +85,8 @@ struct PosSrc {
 DN_DEVINL uint32_t pos_of(const PosSrc& s) { return s.sp ? s.sp->pos : s.pos; }
 
 // ---- embedding -----------------------------------------------------------------------------------------------------
-// x[t] = embed[token] + bigram[(prev * mul_prev + token * mul_cur) mod buckets]; the first token of a sequence takes the
-// extra row `buckets`.  The token history lives on the device (tokens[position]): the previous token of a portion's
+// x[t] = (embed[token] + bigram[(prev * mul_prev + token * mul_cur) mod buckets]) * scale; the first token of a sequence takes
+// the extra row `buckets`.  The token history lives on the device (tokens[position]): the previous token of a portion's
 // first row is whatever the previous step left there.
 template <typename WT> struct EmbedRowsParams {
     const WT* embed; const WT* bigram;   // bigram may be null
@@ -93,6 +94,8 @@ template <typename WT> struct EmbedRowsParams {
     float* x; int width;
     PosSrc ps;
     uint32_t buckets, mul_prev, mul_cur;
+    float scale = 1.0f;
+    WT* h = nullptr;                     // when set: x again in the operand type (a sublayer that reads the embedding unnormed)
 };
 template <typename WT> __global__ void __launch_bounds__(128) embed_rows_kernel(const EmbedRowsParams<WT> p) {
     pdl_launch();
@@ -112,7 +115,11 @@ template <typename WT> __global__ void __launch_bounds__(128) embed_rows_kernel(
         b = p.bigram + (size_t)row * p.width;
     }
     float* x = p.x + (size_t)t * p.width;
-    for (int c = threadIdx.x; c < p.width; c += blockDim.x) x[c] = to_f(e[c]) + (b ? to_f(b[c]) : 0.0f);
+    for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+        const float v = (to_f(e[c]) + (b ? to_f(b[c]) : 0.0f)) * p.scale;
+        x[c] = v;
+        if (p.h) from_f(p.h[(size_t)t * p.width + c], v);
+    }
 }
 
 // ---- RMS norm of rows -----------------------------------------------------------------------------------------------
@@ -243,22 +250,35 @@ template <typename AT> __global__ void __launch_bounds__(256) layernorm_rows_ker
 // (without wb the row is x itself), then with w_next the next sublayer's input
 //     g[c] = x[c] / sqrt(mean(x^2) + eps) * w_next[c];      h[c] = g[c] + (before[c] - g[c]) * mu[c]        (mu: token shift)
 // where `before` is the previous token's g: read from prev (zeros when `fresh`, the first token of a sequence), which then takes
-// this token's g.  inv_out asks for the factor 1 / sqrt(mean(x^2) + eps) instead of h.  Rows up to CACHE * blockDim.x columns stay
-// in registers; longer ones are loaded again.  EARLY: the weights are loaded with the row instead of when they are needed (a single
-// row is nothing but latency).
-template <typename AT, int CACHE, bool EARLY>
-DN_DEVINL void sandwich_row(const float* y, int n, float* x, const float* wb, float eps, float* red, const float* w_next, const float* mu, float* prev,
+// this token's g.  h without w_next: h[c] = x[c] (the next sublayer reads the residual row itself).  inv_out asks for the factor
+// 1 / sqrt(mean(x^2) + eps) instead of h.  y comes from `src`: src.fill(v) loads this thread's columns at once, src.at(c) one of them
+// (a plain row, or something computed per column).  Rows up to CACHE * blockDim.x columns stay in registers; longer ones are loaded
+// again.  EARLY: the weights are loaded with the row instead of when they are needed (a single row is nothing but latency).
+struct PlainRow {
+    const float* y; int n;
+    template <int CACHE> DN_DEVINL void fill(float (&v)[CACHE]) const {
+#pragma unroll
+        for (int i = 0; i < CACHE; i++) {
+            const int c = threadIdx.x + i * blockDim.x;
+            v[i] = c < n ? y[c] : 0.0f;
+        }
+    }
+    DN_DEVINL float at(int c) const { return y[c]; }
+};
+template <typename AT, int CACHE, bool EARLY, typename SRC>
+DN_DEVINL void sandwich_row(const SRC& src, int n, float* x, const float* wb, float eps, float* red, const float* w_next, const float* mu, float* prev,
                             bool fresh, AT* h, float* inv_out) {
-    const bool cached = n <= CACHE * (int)blockDim.x;
+    const bool cached = n <= CACHE * (int)blockDim.x, plain = h && !w_next;
     float v[CACHE];
     float wv[EARLY ? CACHE : 1], mv[EARLY ? CACHE : 1], pv[EARLY ? CACHE : 1];
     float ss = 0.0f;
     if (cached) {
         float xv[CACHE], bv[EARLY ? CACHE : 1];
+        if (wb) src.fill(v);
 #pragma unroll
         for (int i = 0; i < CACHE; i++) {
             const int c = threadIdx.x + i * blockDim.x;
-            v[i] = c < n ? (wb ? y[c] : x[c]) : 0.0f;
+            if (!wb) v[i] = c < n ? x[c] : 0.0f;
             xv[i] = c < n && wb ? x[c] : 0.0f;
             if (EARLY) {
                 bv[i] = c < n && wb ? wb[c] : 0.0f;
@@ -279,13 +299,29 @@ DN_DEVINL void sandwich_row(const float* y, int n, float* x, const float* wb, fl
                 ss = fmaf(v[i], v[i], ss);
             }
         }
+        if (plain) {
+#pragma unroll
+            for (int i = 0; i < CACHE; i++) {
+                const int c = threadIdx.x + i * blockDim.x;
+                if (c < n) from_f(h[c], v[i]);
+            }
+        }
     } else if (wb) {
-        for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(y[c], y[c], ss);
+        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = src.at(c); ss = fmaf(a, a, ss); }
         const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
         ss = 0.0f;
-        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float a = x[c] + y[c] * inv * wb[c]; x[c] = a; ss = fmaf(a, a, ss); }
+        for (int c = threadIdx.x; c < n; c += blockDim.x) {
+            const float a = x[c] + src.at(c) * inv * wb[c];
+            x[c] = a;
+            ss = fmaf(a, a, ss);
+            if (plain) from_f(h[c], a);
+        }
     } else {
-        for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
+        for (int c = threadIdx.x; c < n; c += blockDim.x) {
+            const float a = x[c];
+            ss = fmaf(a, a, ss);
+            if (plain) from_f(h[c], a);
+        }
     }
     if (!w_next && !inv_out) return;
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps);
@@ -317,7 +353,7 @@ DN_DEVINL void sandwich_row(const float* y, int n, float* x, const float* wb, fl
 template <typename AT> struct ResNormRowsParams {
     const float* y; int ldy; const float* wb;      // wb null: no sublayer output
     float* x; int ldx; int n; float eps;
-    const float* w_next; AT* h; int ldh;           // or null
+    const float* w_next; AT* h; int ldh;           // or null (h without w_next: the residual row itself)
     const float* mu; float* prev;                  // one row only: the shift here
     float* inv_out;                                // [T]: many rows: the factors for norm_shift_rows_kernel
     PosSrc ps;
@@ -328,7 +364,7 @@ template <typename AT, bool ONE> __global__ void __launch_bounds__(ONE ? 1024 : 
     pdl_launch();
     pdl_wait();
     const int r = blockIdx.x;
-    sandwich_row<AT, ONE ? 4 : 12, ONE>(p.wb ? p.y + (size_t)r * p.ldy : nullptr, p.n, p.x + (size_t)r * p.ldx, p.wb, p.eps, red, p.w_next, p.mu, p.prev,
+    sandwich_row<AT, ONE ? 4 : 12, ONE>(PlainRow{p.wb ? p.y + (size_t)r * p.ldy : nullptr, p.n}, p.n, p.x + (size_t)r * p.ldx, p.wb, p.eps, red, p.w_next, p.mu, p.prev,
                                         p.mu && pos_of(p.ps) == 0, p.h ? p.h + (size_t)r * p.ldh : nullptr, p.inv_out ? p.inv_out + r : nullptr);
 }
 // g_t = x_t * inv[t] * w;  h_t = g_t + (g_{t-1} - g_t) * mu.  Row -1 is prev_in (zeros for a step at position 0); the last row's g
@@ -493,7 +529,7 @@ template <typename AT> struct EpiParams {
     float scale;
     const float* ls;
     AT* act; int lda;         // EPI_GLU: act = glu(gate, up) in the operand type;  EPI_ACT: act = f(acc)
-    const float* bias;        // EPI_STORE: optional bias of the projection
+    const float* bias;        // EPI_STORE, EPI_ACT: optional bias of the projection (EPI_ACT: before the activation)
     const float* tanh_alpha;  // EPI_RESID: when set, f(acc) = tanh(*tanh_alpha * acc) (a tanh norm on the way into the residual)
     const float* lb;          // EPI_RESID: optional shift
     int glu_kind;             // EPI_GLU: GLU_SILU silu(gate) * up | GLU_CLAMPED g = min(gate, limit), u = clamp(up, +-limit):
@@ -525,7 +561,7 @@ template <int EPI, typename AT> DN_DEVINL void epi_apply(const EpiParams<AT>& e,
         e.out[(size_t)t * e.ldo + o] += e.lb ? e.ls[o] * a + e.lb[o] : e.ls[o] * a;
     }
     else if (EPI == EPI_GLU) from_f(e.act[(size_t)t * e.lda + o], glu_apply(e, a, b));
-    else from_f(e.act[(size_t)t * e.lda + o], act_apply(e, a));
+    else from_f(e.act[(size_t)t * e.lda + o], act_apply(e, e.bias ? a + e.bias[o] : a));
 }
 
 // ---- one row times a matrix: W [O][K] streamed once ----------------------------------------------------------------------
@@ -536,7 +572,8 @@ template <int EPI, typename AT> DN_DEVINL void epi_apply(const EpiParams<AT>& e,
 //   NORM_LAYER (x - mean) * rsqrt(var + eps) * nw
 // Batch (gridDim.y > 1): CTA row y multiplies input a + y * a_bs by matrix w + bidx[y] * w_bs (bidx null: y itself) and
 // writes at out/act + y * o_bs -- one matrix per head, or the experts a router picked, read from its device-side list.  A
-// list entry >= n_mats (when n_mats > 0) names an expert without matrices: its CTAs leave at once.
+// list entry >= n_mats (when n_mats > 0) names an expert without matrices: its CTAs leave at once.  With `extra.w` the last CTA row
+// multiplies a matrix of its own (its input, sizes and output may differ from the batch's: a shared expert beside the chosen ones).
 enum { NORM_NONE = 0, NORM_RMS = 1, NORM_TANH = 2, NORM_LAYER = 3 };
 // What follows an EPI_STORE product whose whole output row is a sublayer's result (ln.counter set): the CTA that finishes last
 // -- every CTA takes a ticket from *counter after its stores -- sends the row e.out[0 .. O) through a layer norm into the
@@ -546,6 +583,11 @@ template <typename AT> struct LnTail {
     unsigned int* counter;
     const float* w; const float* ls; float eps;
     float* x; AT* h;
+};
+template <typename AT, typename WT> struct GemvExtra {
+    const AT* a; const WT* w; const WT* w2;
+    int K, O;
+    float* out; AT* act;
 };
 template <typename AT, typename WT> struct GemvRowsParams {
     const AT* a;              // [K] input row (NORM_NONE)
@@ -558,6 +600,7 @@ template <typename AT, typename WT> struct GemvRowsParams {
     EpiParams<AT> e;
     const int* bidx; long long a_bs, w_bs, o_bs;
     int n_mats;
+    GemvExtra<AT, WT> extra;
     LnTail<AT> ln;
 };
 template <typename WT> struct Vec16;
@@ -629,9 +672,11 @@ template <typename AT, typename WT, int EPI, int NORM>
 static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsParams<AT, WT> pp) {
     extern __shared__ __align__(16) float gv_xs[];   // [K rounded up to 4] the input row as f32, then reduction slots
     GemvRowsParams<AT, WT> p = pp;
-    float* red = gv_xs + ((p.K + 3) & ~3);
     pdl_launch();
-    if (gridDim.y > 1 || p.bidx) {   // the expert list is written by the step's router kernel: read it after the wait
+    if (p.extra.w && blockIdx.y == gridDim.y - 1) {
+        p.a = p.extra.a; p.w = p.extra.w; p.w2 = p.extra.w2; p.K = p.extra.K; p.O = p.extra.O; p.e.out = p.extra.out; p.e.act = p.extra.act;
+        p.ksplit = p.ksplit && p.K % Vec16<WT>::N == 0;
+    } else if (gridDim.y > 1 || p.bidx) {   // the expert list is written by the step's router kernel: read it after the wait
         if (p.bidx) pdl_wait();
         const long long by = blockIdx.y, bw = p.bidx ? p.bidx[by] : by;
         if (p.n_mats > 0 && bw >= p.n_mats) return;
@@ -641,6 +686,7 @@ static __global__ void __launch_bounds__(256) gemv_rows_kernel(const GemvRowsPar
         if (p.e.out) p.e.out += by * p.o_bs;
         if (p.e.act) p.e.act += by * p.o_bs;
     }
+    float* red = gv_xs + ((p.K + 3) & ~3);
     if (p.pdl) {   // weights do not depend on the predecessor: ask L2 for this warp's first rows while waiting for it
         const int w0 = (int)(blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5));
         const int o = p.ksplit ? 2 * (int)blockIdx.x : (EPI == EPI_GLU ? w0 : 2 * w0);

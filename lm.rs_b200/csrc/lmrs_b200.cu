@@ -1459,7 +1459,7 @@ extern "C" void lmrs_b200_destroy(lmrs_b200_t* m) {
 }
 
 // ---- models that come as a folder (config.json + model.safetensors): arch.h ----------------------------------------------
-namespace lmrs { void register_genetar(); void register_tudatar(); void register_rupenex(); void register_badepel(); void register_bolapel(); }
+namespace lmrs { void register_genetar(); void register_tudatar(); void register_rupenex(); void register_badepel(); void register_bolapel(); void register_lutesun(); }
 static void register_architectures() {
     static bool done = false;
     if (done) return;
@@ -1469,6 +1469,7 @@ static void register_architectures() {
     register_rupenex();
     register_badepel();
     register_bolapel();
+    register_lutesun();
 }
 static int open_arch(const char* dir, int device, int dtype, uint32_t max_tokens, lmrs_b200_t** out) {
     int ndev = 0;

@@ -1,7 +1,8 @@
 // mixer_ops.cuh -- what happens between a sequence mixer's input projection and its core, for the mixers that are not plain
 // multi-head attention, and the one core that is not attention (dense_ops.cuh has the attention kernel):
-//   latent_kv_post_kernel     attention through a shared latent: RMS norm of the query latent and of the key/value latent,
-//                             pairwise rotation of the shared rotated key part, latent + rotated part written to the cache
+//   latent_kv_post_kernel     attention through a shared latent: RMS norm of the query latent (when there is one) and of the
+//                             key/value latent, rotation of the shared rotated key part (neighbouring pairs or halves), latent +
+//                             rotated part written to the cache, sigmoid of per-head output gate logits
 //   latent_q_post_kernel      per query head: unrotated part to the operand type (it is multiplied into the latent space
 //                             next), rotated part rotated and placed behind the latent-space part of the query; or, for the
 //                             per-head form, the whole head [unrotated | rotated] in f32
@@ -44,15 +45,37 @@ DN_DEVINL void rotate_pairs_warp(const float* src, float* dst, int n, int rot_di
     for (int d = rot_dims + lane; d < n; d += 32) dst[d] = src[d];
 }
 
-// ---- attention through a latent: the projected row [query latent (rq) | key/value latent (rk) | rotated key part (dr)] ----
+// the same with dimension i turned together with i + rot_dims/2
+DN_DEVINL void rotate_halves_warp(const float* src, float* dst, int n, int rot_dims, const float* c, const float* s, int lane) {
+    const int half = rot_dims / 2;
+    for (int i = lane; i < half; i += 32) {
+        const float u = src[i], v = src[i + half];
+        dst[i] = u * c[i] - v * s[i];
+        dst[i + half] = v * c[i] + u * s[i];
+    }
+    for (int d = rot_dims + lane; d < n; d += 32) dst[d] = src[d];
+}
+struct Rotation {
+    int dims, halves;                          // halves: pairs (i, i + dims/2) instead of (2i, 2i+1)
+    const float* cos; const float* sin;        // [max_tokens][dims/2], a multiplier folded in
+};
+DN_DEVINL void rotate_warp(const Rotation& r, uint32_t pos, const float* src, float* dst, int n, int lane) {
+    const float *c = r.cos + (size_t)pos * (r.dims / 2), *s = r.sin + (size_t)pos * (r.dims / 2);
+    if (r.halves) rotate_halves_warp(src, dst, n, r.dims, c, s, lane);
+    else rotate_pairs_warp(src, dst, n, r.dims, c, s, lane);
+}
+
+// ---- attention through a latent: the projected row holds [key/value latent (rk) | rotated key part (dr)] at column kv_off and may
+// hold a query latent (rq) at column 0 and output gate logits (one per head) at column gate_off -------------------------------
 template <typename AT> struct LatentKvPostParams {
     const float* in; int ld;
-    int rq, rk, dr;
+    int rq, kv_off, rk, dr;                                       // rq == 0: no query latent
     const float* wq; const float* wkv; float eps;                 // norm weights of the two latents
-    int rot_dims; const float* rot_cos; const float* rot_sin;      // [max_tokens][rot_dims/2], multiplier folded in
+    Rotation rot;
     AT* cq_out;                                                   // [T][rq]
     float* cache;                                                 // [max_tokens][rk + dr]
     AT* cache_op;                                                 // [max_tokens][rk]: the latent again, in the operand type
+    float* gate_out; int H, gate_off;                             // or null: [T][H] sigmoid(gate logit)
     PosSrc ps;
 };
 template <typename AT> __global__ void __launch_bounds__(256) latent_kv_post_kernel(const LatentKvPostParams<AT> p) {
@@ -62,12 +85,16 @@ template <typename AT> __global__ void __launch_bounds__(256) latent_kv_post_ker
     const int t = blockIdx.x;
     const uint32_t pos = pos_of(p.ps) + (uint32_t)t;
     const float* row = p.in + (size_t)t * p.ld;
-    float ss = 0.0f;
-    for (int c = threadIdx.x; c < p.rq; c += blockDim.x) ss += row[c] * row[c];
-    ss = block_sum(ss, red);
-    float inv = 1.0f / sqrtf(ss / (float)p.rq + p.eps);
-    for (int c = threadIdx.x; c < p.rq; c += blockDim.x) from_f(p.cq_out[(size_t)t * p.rq + c], row[c] * inv * p.wq[c]);
-    const float* kv = row + p.rq;
+    float ss = 0.0f, inv;
+    if (p.rq > 0) {
+        for (int c = threadIdx.x; c < p.rq; c += blockDim.x) ss += row[c] * row[c];
+        ss = block_sum(ss, red);
+        inv = 1.0f / sqrtf(ss / (float)p.rq + p.eps);
+        for (int c = threadIdx.x; c < p.rq; c += blockDim.x) from_f(p.cq_out[(size_t)t * p.rq + c], row[c] * inv * p.wq[c]);
+    }
+    if (p.gate_out)
+        for (int h = threadIdx.x; h < p.H; h += blockDim.x) p.gate_out[(size_t)t * p.H + h] = 1.0f / (1.0f + expf(-row[p.gate_off + h]));
+    const float* kv = row + p.kv_off;
     ss = 0.0f;
     for (int c = threadIdx.x; c < p.rk; c += blockDim.x) ss += kv[c] * kv[c];
     ss = block_sum(ss, red);
@@ -78,16 +105,13 @@ template <typename AT> __global__ void __launch_bounds__(256) latent_kv_post_ker
         dst[c] = v;
         from_f(p.cache_op[(size_t)pos * p.rk + c], v);
     }
-    if (threadIdx.x < 32) {
-        const int half = p.rot_dims / 2;
-        rotate_pairs_warp(kv + p.rk, dst + p.rk, p.dr, p.rot_dims, p.rot_cos + (size_t)pos * half, p.rot_sin + (size_t)pos * half, threadIdx.x);
-    }
+    if (threadIdx.x < 32) rotate_warp(p.rot, pos, kv + p.rk, dst + p.rk, p.dr, threadIdx.x);
 }
 
 template <typename AT> struct LatentQPostParams {
-    const float* q;           // [T][H * (dn + dr)], head by head [unrotated | rotated]
+    const float* q; int ldq;  // [T][H * (dn + dr)] in rows of ldq floats, head by head [unrotated | rotated]
     int H, dn, dr, rk;
-    int rot_dims; const float* rot_cos; const float* rot_sin;
+    Rotation rot;
     AT* qn_out;               // [T][H * dn]
     float* qabs;              // [T][H * (rk + dr)]: the rotated part goes to columns rk .. rk+dr of each head
     float* qfull;             // when set instead: [T][H * (dn + dr)], the unrotated part copied, the rotated part rotated
@@ -100,31 +124,29 @@ template <typename AT> __global__ void __launch_bounds__(128) latent_q_post_kern
     const int h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (h >= p.H) return;
     const uint32_t pos = pos_of(p.ps) + (uint32_t)t;
-    const float* src = p.q + ((size_t)t * p.H + h) * (p.dn + p.dr);
-    const int half = p.rot_dims / 2;
+    const float* src = p.q + (size_t)t * p.ldq + (size_t)h * (p.dn + p.dr);
     if (p.qfull) {
         float* dst = p.qfull + ((size_t)t * p.H + h) * (p.dn + p.dr);
         for (int d = lane; d < p.dn; d += 32) dst[d] = src[d];
-        rotate_pairs_warp(src + p.dn, dst + p.dn, p.dr, p.rot_dims, p.rot_cos + (size_t)pos * half, p.rot_sin + (size_t)pos * half, lane);
+        rotate_warp(p.rot, pos, src + p.dn, dst + p.dn, p.dr, lane);
         return;
     }
     AT* qn = p.qn_out + ((size_t)t * p.H + h) * p.dn;
     for (int d = lane; d < p.dn; d += 32) from_f(qn[d], src[d]);
-    rotate_pairs_warp(src + p.dn, p.qabs + ((size_t)t * p.H + h) * (p.rk + p.dr) + p.rk, p.dr, p.rot_dims,
-                      p.rot_cos + (size_t)pos * half, p.rot_sin + (size_t)pos * half, lane);
+    rotate_warp(p.rot, pos, src + p.dn, p.qabs + ((size_t)t * p.H + h) * (p.rk + p.dr) + p.rk, p.dr, lane);
 }
 
-// keys per head for positions 0 .. n: kfull[j][h] = [knope[j][h] (dn) | cached rotated part of position j (dr)]
+// keys per head for positions j0 .. j0 + gridDim.x: kfull[j][h] = [knope[j][h] (dn) | cached rotated part of position j (dr)]
 struct LatentExpandParams {
     const float* knope;       // [n][H * dn] up-projected latents
     const float* cache;       // [max_tokens][rk + dr]
     float* kfull;             // [n][H * (dn + dr)]
-    int H, dn, dr, rk;
+    int H, dn, dr, rk, j0;
 };
 static __global__ void __launch_bounds__(256) latent_expand_kernel(const LatentExpandParams p) {
     pdl_launch();
     pdl_wait();
-    const int j = blockIdx.x, dq = p.dn + p.dr;
+    const int j = p.j0 + (int)blockIdx.x, dq = p.dn + p.dr;
     const float* kr = p.cache + (size_t)j * (p.rk + p.dr) + p.rk;
     for (int e = threadIdx.x; e < p.H * dq; e += blockDim.x) {
         const int h = e / dq, d = e - h * dq;

@@ -1,7 +1,9 @@
 // moe_ops.cuh -- a feed-forward made of routed experts, around the matrix kernels of dense_ops.cuh / dense_gemm.cuh:
-//   moe_logits_kernel    router logits in f32 (f32 router matrix)
+//   moe_logits_kernel    router logits in f32 (f32 router matrix), and the logits of further rows stacked below the router's (a
+//                        gate on a shared expert)
 //   moe_topk_kernel      score = sigmoid(logit), or the softmax over all logits; the `top` experts with the largest
-//                        score + correction[e] are chosen, their weights are score / (sum of chosen scores + 1e-20) * scale
+//                        score + correction[e] are chosen, their weights are score / (sum of chosen scores + 1e-20) * scale; the
+//                        choice may be limited to the best `keep` of `groups` equal groups of neighbouring experts
 //   moe_sort_kernel      (token, choice) pairs counted and sorted by expert: row offsets per expert, the slot of every pair,
 //                        the token of every slot
 //   moe_gather_kernel    the normalised rows copied into expert order (the grouped matrix kernels then see one contiguous row
@@ -9,9 +11,10 @@
 //   moe_combine_kernel   x += f(sum over the token's choices of weight * expert output), f = a tanh norm on the way into the
 //                        residual (or the identity); or the sum stored for a norm that needs statistics.  Experts beyond
 //                        the ones with matrices are identity experts (their output is the token's input row); a shared
-//                        expert's output row can be added
+//                        expert's output row can be added, times the sigmoid of one logit per token
 //   moe_combine_layernorm_kernel   the same sum through a layer norm into the residual stream: one CTA per token, or a
 //                        single token's columns over several CTAs of which the last one to finish applies the norm
+//   moe_combine_resnorm_kernel     the same sum through an RMS norm into the residual stream (resnorm_rows_kernel's row pass)
 // A one-row step needs no sorting: the one-row matrix kernel takes the chosen experts from the router's device-side list.
 #pragma once
 #include "dense_ops.cuh"
@@ -25,11 +28,14 @@ template <typename AT> struct MoeRouterParams {
     const float* router;          // [E][width]
     const float* correction;      // [E], added for the choice only
     int E, top, width;
+    int extra;                    // further rows of `router` (behind the E) whose logits are computed with it and never chosen
+    int groups, keep;             // groups > 1: E / groups neighbouring outputs form a group that scores its largest choice score;
+                                  // only the `keep` best groups can be chosen from (keep * (E / groups) >= top)
     int softmax;                  // 0: score = sigmoid(logit); 1: scores = softmax over the E logits; 2: the largest logits are
                                   // chosen and the weights are the softmax over the chosen logits only (times scale)
     const float* bias;            // [E] or null: added to the router logits
     float scale;
-    float* z;                     // [T][E] router logits (scratch between the two kernels)
+    float* z;                     // [T][E + extra] router logits (scratch between the two kernels)
     int* idx; float* wts;         // [T][top]
 };
 // logits: one warp per (token, expert), so that a single token still spreads over E warps on many SMs
@@ -38,7 +44,8 @@ template <typename AT> __global__ void __launch_bounds__(128) moe_logits_kernel(
     pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int e = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (e >= p.E) return;
+    const int rows = p.E + p.extra;
+    if (e >= rows) return;
     const float* w = p.router + (size_t)e * p.width;
     float a = 0.0f;
     if (p.h) {
@@ -52,30 +59,48 @@ template <typename AT> __global__ void __launch_bounds__(128) moe_logits_kernel(
         for (int c = lane; c < p.width; c += 32) { AT r; from_f(r, tanhnorm_apply(p.tn, alpha, c, x[c])); a = fmaf(w[c], to_f(r), a); }
     }
     a = warp_sum(a);
-    if (lane == 0) p.z[(size_t)t * p.E + e] = p.bias ? a + p.bias[e] : a;
+    if (lane == 0) p.z[(size_t)t * rows + e] = p.bias && e < p.E ? a + p.bias[e] : a;
 }
 // choice: one warp per token
 template <typename AT> __global__ void __launch_bounds__(32) moe_topk_kernel(const MoeRouterParams<AT> p) {
     extern __shared__ __align__(16) float mr_sm[];
     float* score = mr_sm;            // [E] sigmoid(logit)
-    float* choice = score + p.E;     // [E] score + correction; -inf once chosen
+    float* choice = score + p.E;     // [E] score + correction; -inf once chosen or when its group is out
+    float* gscore = choice + p.E;    // [groups] (groups > 1)
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x;
+    const float* zt = p.z + (size_t)t * (p.E + p.extra);
     float zmax = -INFINITY, zsum = 0.0f;
     if (p.softmax == 1) {
-        for (int e = lane; e < p.E; e += 32) zmax = fmaxf(zmax, p.z[(size_t)t * p.E + e]);
+        for (int e = lane; e < p.E; e += 32) zmax = fmaxf(zmax, zt[e]);
         zmax = warp_max(zmax);
-        for (int e = lane; e < p.E; e += 32) zsum += expf(p.z[(size_t)t * p.E + e] - zmax);
+        for (int e = lane; e < p.E; e += 32) zsum += expf(zt[e] - zmax);
         zsum = warp_sum(zsum);
     }
     for (int e = lane; e < p.E; e += 32) {
-        const float z = p.z[(size_t)t * p.E + e];
+        const float z = zt[e];
         const float sg = p.softmax == 2 ? z : (p.softmax == 1 ? expf(z - zmax) / zsum : 1.0f / (1.0f + expf(-z)));
         score[e] = sg;
         choice[e] = sg + (p.correction ? p.correction[e] : 0.0f);
     }
     __syncwarp();
+    if (p.groups > 1) {
+        const int size = p.E / p.groups;
+        for (int g = lane; g < p.groups; g += 32) {
+            float m = choice[g * size];
+            for (int i = 1; i < size; i++) m = fmaxf(m, choice[g * size + i]);
+            gscore[g] = m;
+        }
+        __syncwarp();
+        for (int g = lane; g < p.groups; g += 32) {   // a group stays when fewer than `keep` others are better (a tie: the lower index)
+            int better = 0;
+            for (int o = 0; o < p.groups; o++) better += gscore[o] > gscore[g] || (gscore[o] == gscore[g] && o < g) ? 1 : 0;
+            if (better >= p.keep)
+                for (int i = 0; i < size; i++) choice[g * size + i] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float sum = 0.0f;
     for (int k = 0; k < p.top; k++) {
         float best = -INFINITY;
@@ -88,6 +113,7 @@ template <typename AT> __global__ void __launch_bounds__(32) moe_topk_kernel(con
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
+        if (bi >= p.E) bi = k;   // scores that are no numbers compare with nothing: stay inside the list
         const float sg = score[bi];
         sum += sg;
         if (lane == 0) { p.idx[(size_t)t * p.top + k] = bi; p.wts[(size_t)t * p.top + k] = sg; choice[bi] = -INFINITY; }
@@ -157,12 +183,14 @@ struct MoeCombineParams {
     int top, width;
     const int* idx; int n_real;        // idx set: a pair whose expert idx[t][k] >= n_real is an identity expert ...
     const float* xin; int ld_in;       // ... whose output is row t of xin
-    const float* add;                  // or null: [T][width] added to the sum (a shared expert's output)
+    const float* add;                  // or null: [T][width] added to the sum (a shared expert's output) ...
+    const float* add_gate; int ld_gate;   // ... times sigmoid(add_gate[t * ld_gate]) when set
     float* out; int ldo;               // when set: the sum is stored here and x is left alone
 };
-// the weighted sum of one token's expert outputs at column c
-DN_DEVINL float moe_combined(const MoeCombineParams& p, int t, int c) {
-    float a = p.add ? p.add[(size_t)t * p.width + c] : 0.0f;
+DN_DEVINL float moe_add_gate(const MoeCombineParams& p, int t) { return p.add_gate ? 1.0f / (1.0f + expf(-p.add_gate[(size_t)t * p.ld_gate])) : 1.0f; }
+// the weighted sum of one token's expert outputs at column c; ag = moe_add_gate of the token
+DN_DEVINL float moe_combined(const MoeCombineParams& p, int t, int c, float ag = 1.0f) {
+    float a = p.add ? ag * p.add[(size_t)t * p.width + c] : 0.0f;
     for (int k = 0; k < p.top; k++) {
         const float w = p.wts[(size_t)t * p.top + k];
         if (p.idx && p.idx[(size_t)t * p.top + k] >= p.n_real) { a = fmaf(w, p.xin[(size_t)t * p.ld_in + c], a); continue; }
@@ -175,9 +203,9 @@ static __global__ void __launch_bounds__(256) moe_combine_kernel(const MoeCombin
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
-    const float alpha = p.n.alpha ? *p.n.alpha : 0.0f;
+    const float alpha = p.n.alpha ? *p.n.alpha : 0.0f, ag = moe_add_gate(p, t);
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < p.width; c += gridDim.y * blockDim.x) {
-        const float a = moe_combined(p, t, c);
+        const float a = moe_combined(p, t, c, ag);
         if (p.out) p.out[(size_t)t * p.ldo + c] = a;
         else p.x[(size_t)t * p.ldx + c] += p.n.alpha ? tanhnorm_apply(p.n, alpha, c, a) : a;
     }
@@ -200,12 +228,13 @@ template <typename AT> __global__ void __launch_bounds__(256) moe_combine_layern
     pdl_wait();
     const int t = blockIdx.x;
     float* xr = p.c.x + (size_t)t * p.c.ldx;
+    const float ag = moe_add_gate(p.c, t);
     if (gridDim.y == 1) {
-        layernorm_row<AT>([&](int c) { return moe_combined(p.c, t, c); }, p.c.width, p.w, p.eps, red, xr, p.ls, nullptr, p.h + (size_t)t * p.ldh);
+        layernorm_row<AT>([&](int c) { return moe_combined(p.c, t, c, ag); }, p.c.width, p.w, p.eps, red, xr, p.ls, nullptr, p.h + (size_t)t * p.ldh);
         return;
     }
     float* row = p.c.out + (size_t)t * p.c.ldo;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < p.c.width; c += gridDim.y * blockDim.x) row[c] = moe_combined(p.c, t, c);
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < p.c.width; c += gridDim.y * blockDim.x) row[c] = moe_combined(p.c, t, c, ag);
     __threadfence();   // this thread's stores of the row before the ticket
     __syncthreads();
     if (threadIdx.x == 0) last = atomicAdd(p.counter, 1u) == gridDim.y - 1 ? 1u : 0u;
@@ -214,6 +243,56 @@ template <typename AT> __global__ void __launch_bounds__(256) moe_combine_layern
     __threadfence();
     layernorm_row<AT>([&](int c) { return __ldcg(row + c); }, p.c.width, p.w, p.eps, red, xr, p.ls, nullptr, p.h + (size_t)t * p.ldh);
     if (threadIdx.x == 0) *p.counter = 0u;
+}
+
+// the same sum sent through an RMS norm into the residual stream, x <- x + rms(sum) w, with x again in the operand type to h: one CTA
+// per token (ONE: a single token, up to 1024 threads).  A thread loads its columns of several experts before it adds the first.
+struct MoeRow {
+    const MoeCombineParams& p;
+    int t;
+    float ag;
+    template <int CACHE> DN_DEVINL void fill(float (&v)[CACHE]) const {
+        constexpr int KU = CACHE <= 4 ? 4 : 1;   // experts in flight
+#pragma unroll
+        for (int i = 0; i < CACHE; i++) {
+            const int c = threadIdx.x + i * blockDim.x;
+            v[i] = p.add && c < p.width ? ag * p.add[(size_t)t * p.width + c] : 0.0f;
+        }
+        for (int k0 = 0; k0 < p.top; k0 += KU) {
+            float w[KU], e[KU][CACHE];
+#pragma unroll
+            for (int u = 0; u < KU; u++) {
+                const int k = min(k0 + u, p.top - 1);
+                const size_t pair = (size_t)t * p.top + k;
+                w[u] = k0 + u < p.top ? p.wts[pair] : 0.0f;
+                const float* row = p.idx && p.idx[pair] >= p.n_real ? p.xin + (size_t)t * p.ld_in : p.y + (p.slot ? (size_t)p.slot[pair] : pair) * p.width;
+#pragma unroll
+                for (int i = 0; i < CACHE; i++) {
+                    const int c = threadIdx.x + i * blockDim.x;
+                    e[u][i] = c < p.width ? row[c] : 0.0f;
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < KU; u++)
+#pragma unroll
+                for (int i = 0; i < CACHE; i++)
+                    if (k0 + u < p.top) v[i] = fmaf(w[u], e[u][i], v[i]);
+        }
+    }
+    DN_DEVINL float at(int c) const { return moe_combined(p, t, c, ag); }
+};
+template <typename AT> struct MoeCombineResNormParams {
+    MoeCombineParams c;
+    const float* w; float eps;
+    AT* h; int ldh;
+};
+template <typename AT, bool ONE> __global__ void __launch_bounds__(ONE ? 1024 : 256) moe_combine_resnorm_kernel(const MoeCombineResNormParams<AT> p) {
+    __shared__ float red[33];
+    pdl_launch();
+    pdl_wait();
+    const int t = blockIdx.x;
+    sandwich_row<AT, ONE ? 4 : 16, ONE>(MoeRow{p.c, t, moe_add_gate(p.c, t)}, p.c.width, p.c.x + (size_t)t * p.c.ldx, p.w, p.eps, red, nullptr, nullptr, nullptr,
+                                        false, p.h + (size_t)t * p.ldh, nullptr);
 }
 
 }  // namespace dense

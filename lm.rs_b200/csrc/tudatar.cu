@@ -6,11 +6,7 @@
 //                       and key channel from a low-rank projection, state S [dk][dv] per head in f32, output RMS-normed per
 //                       head and gated by a second low-rank projection
 //   "latent_attention"  softmax attention whose keys and values are up-projections of one cached latent per token plus one
-//                       rotated key part shared by all heads; queries go through a latent of their own.  Short steps run in
-//                       the latent space: the up-projection of the keys is multiplied into the query, the attention kernel
-//                       sees one shared key/value head of size kv_rank (+ rot_dim), and the values' up-projection follows it.
-//                       Long portions up-project all cached latents to per-head keys and values first (tensor cores) and run
-//                       ordinary multi-head attention over them: a third of the attention arithmetic
+//                       rotated key part shared by all heads; queries go through a latent of their own (latent_mixer.cuh)
 //   "attention"         grouped-head attention with projection biases, q and k RMS-normed over the whole projection, values
 //                       normed per head, a sliding window and a logarithmic distance penalty per head, no rotation
 // and a feed-forward of routed experts (sigmoid router, choice with a correction, normalised weights).  logits =
@@ -18,8 +14,7 @@
 // the generic ones of dense_ops.cuh / mixer_ops.cuh / moe_ops.cuh / dense_gemm.cuh, the step / chunking / graph machinery
 // is DenseModel's.  Caches are addressed by position like those of the other models; the recurrent state and the convolution
 // tails continue from the previous step and restart when a step begins at position 0.
-#include "dense_model.cuh"
-#include "mixer_ops.cuh"
+#include "latent_mixer.cuh"
 #include "moe_ops.cuh"
 
 namespace lmrs {
@@ -65,15 +60,13 @@ struct LayerCfg {
     float scale = 1.0f;
     int window = 0;                       // MIX_WINDOW
     int taps = 0, ra = 0, rg = 0;         // MIX_DELTA
-    int dr = 0, rk = 0, rq = 0;           // MIX_LATENT (dk = unrotated size)
-    bool latent_space_ok = true, per_head_ok = true;
-    RotSpec rot;
+    LatentCfg lat;                        // MIX_LATENT
     MoeCfg moe;
 };
 
-template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, WT> {
+template <typename AT, typename WT> class TudatarModel : public LatentModel<AT, WT> {
   public:
-    typedef DenseModel<AT, WT> B;
+    typedef LatentModel<AT, WT> B;
     using B::load_vec; using B::load_stack; using B::error; using B::launches; using B::info; using B::d_logits; using B::width; using B::vocab; using B::max_tokens;
     using B::sms; using B::d_tokens; using B::cap; using B::x; using B::hn; using B::d_rows; using B::MAX_SPLIT; using B::pdl_now;
     using B::dalloc; using B::dfree; using B::need; using B::upload_w; using B::upload_f32; using B::check_launch; using B::launch_k;
@@ -88,11 +81,7 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
         WT* wo = nullptr;
         // MIX_WINDOW
         float *qnorm = nullptr, *knorm = nullptr, *r1 = nullptr, *r2 = nullptr, *kcache = nullptr, *vcache = nullptr;
-        // MIX_LATENT
-        float *dq_norm = nullptr, *dkv_norm = nullptr, *lcache = nullptr;
-        AT* lcache_op = nullptr;                               // [max_tokens][rk] the latent in the operand type
-        WT *wuq = nullptr, *wuk = nullptr, *wukT = nullptr, *wuv = nullptr;   // wukT: [H][rk][dn], wuk transposed per head
-        const float *rot_cos = nullptr, *rot_sin = nullptr;
+        typename B::Latent lat;                  // MIX_LATENT
         // MIX_DELTA
         float *wconv = nullptr, *tail = nullptr, *a_log = nullptr, *onorm = nullptr, *dt_bias = nullptr, *state = nullptr;
         WT *wa2 = nullptr, *wg2 = nullptr;
@@ -107,13 +96,10 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
     bool has_state = false;      // some layer carries a recurrent state
     uint32_t next_pos = 0;       // where that state stands
     // scratch for `cap` rows
-    AT *h = nullptr, *lat = nullptr, *qn = nullptr, *att = nullptr, *att2 = nullptr, *xg = nullptr, *act = nullptr;
-    float *rz = nullptr, *proj = nullptr, *qa = nullptr, *qb = nullptr, *fa = nullptr, *fb = nullptr, *beta = nullptr, *part = nullptr, *y = nullptr, *wts = nullptr;
+    AT *h = nullptr, *lat = nullptr, *att = nullptr, *xg = nullptr, *act = nullptr;
+    float *rz = nullptr, *proj = nullptr, *qa = nullptr, *fa = nullptr, *fb = nullptr, *beta = nullptr, *part = nullptr, *y = nullptr, *wts = nullptr;
     int *eidx = nullptr, *slot = nullptr, *row_of = nullptr, *grp = nullptr;
-    float *kfull = nullptr, *vfull = nullptr, *knope = nullptr;   // per-head keys and values of all cached positions (long latent-attention portions)
-    int max_kfull = 0, max_vfull = 0, max_knope = 0;
-    int latent_expand_rows = 16;   // portions of at least this many rows take the per-head form
-    int max_proj = 0, max_lat = 0, max_qn = 0, max_att = 0, max_att2 = 0, max_qa = 0, max_qb = 0, max_fa = 0, max_fb = 0, max_H = 0,
+    int max_proj = 0, max_lat = 0, max_att = 0, max_qa = 0, max_fa = 0, max_fb = 0, max_H = 0,
         max_dv = 0, max_top = 0, max_ff = 0, max_E = 0;
 
     size_t n_layers() const override { return layers.size(); }
@@ -135,25 +121,24 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
         } else if (type == "latent_attention") {
             c.kind = MIX_LATENT;
             c.G = 1;
-            c.dr = (int)m.at("rot_dim").number(0); c.rk = (int)m.at("kv_rank").number(0); c.rq = (int)m.at("q_rank").number(0);
-            c.scale = (float)m.at("scale").number(1.0);
-            if (c.dr < 0 || c.rk <= 0 || c.rq <= 0) { error = where + ": rot_dim, kv_rank and q_rank are required"; return 1; }
-            const Json& r = m.at("rot");
-            c.rot.dims = r.is_obj() ? (int)r.at("dims").number(c.dr) : 0;
-            if (c.rot.dims < 0 || c.rot.dims > c.dr || c.rot.dims % 2 != 0) { error = where + ": rot.dims must be even and at most rot_dim"; return 1; }
-            if (r.is_obj()) {
-                c.rot.base = r.at("base").number(10000.0);
+            LatentCfg& l = c.lat;
+            if (this->parse_latent(m, where, l)) return 1;
+            l.rq = (int)m.at("q_rank").number(0);
+            if (l.rq <= 0) { error = where + ": q_rank is required"; return 1; }
+            RotSpec rot;
+            rot.dims = l.rot_dims;
+            if (m.at("rot").is_obj()) {
+                const Json& r = m.at("rot");
+                rot.base = r.at("base").number(10000.0);
                 if (r.has("scaling") && r.at("scaling").is_obj()) {
                     const Json& s = r.at("scaling");
-                    c.rot.scaled = true;
-                    c.rot.factor = s.at("factor").number(1.0); c.rot.fast = s.at("fast").number(32.0);
-                    c.rot.slow = s.at("slow").number(1.0); c.rot.original = s.at("original").number(4096.0);
+                    rot.scaled = true;
+                    rot.factor = s.at("factor").number(1.0); rot.fast = s.at("fast").number(32.0);
+                    rot.slow = s.at("slow").number(1.0); rot.original = s.at("original").number(4096.0);
                 }
             }
-            // a latent too wide for the attention kernel's tiles is always up-projected to per-head keys and values
-            c.latent_space_ok = B::attention_fits(c.rk + c.dr, c.rk);
-            c.per_head_ok = B::attention_fits(c.dk + c.dr, c.dv);
-            if (!c.latent_space_ok && !c.per_head_ok) { error = where + ": neither kv_rank " + std::to_string(c.rk) + " nor the per-head sizes fit the attention kernel's shared-memory tiles"; return 1; }
+            rot.freqs(l.rot_f, l.rot_mult);
+            l.rot_key = rot.key();
         } else if (type == "attention") {
             c.kind = MIX_WINDOW;
             c.G = (int)m.at("kv_heads").number(c.H);
@@ -203,14 +188,6 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
         GCK(cudaMemcpy(*out, host.data(), host.size() * 4, cudaMemcpyHostToDevice));
         return 0;
     }
-    int upload_host(const std::vector<float>& v, WT* dst) {
-        if (std::is_same<WT, float>::value) { GCK(cudaMemcpy(dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice)); return 0; }
-        std::vector<__nv_bfloat16> tmp(v.size());
-        for (size_t i = 0; i < v.size(); i++) tmp[i] = __float2bfloat16_rn(v[i]);
-        GCK(cudaMemcpy(dst, tmp.data(), tmp.size() * 2, cudaMemcpyHostToDevice));
-        return 0;
-    }
-
     int load(const std::string& dir, const Json& cfg, const ArchOptions& opt) {
         sms = opt.sms;
         B::gemm_ctx.sms = opt.sms;
@@ -247,36 +224,9 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
                 max_qa = std::max(max_qa, nq);
                 max_att = std::max(max_att, att_cols);
             } else if (c.kind == MIX_LATENT) {
-                const int dq = c.dk + c.dr;
-                if (load_stack(st, {{q + "dq", c.rq}, {q + "dkv", c.rk + c.dr}}, width, &L.w_in, &L.in_rows)) return 1;
-                if (load_vec(st, q + "dq.norm", c.rq, &L.dq_norm) || load_vec(st, q + "dkv.norm", c.rk, &L.dkv_norm)) return 1;
-                if (load_stack(st, {{q + "uq", c.H * dq}}, c.rq, &L.wuq, nullptr) || load_stack(st, {{q + "uv", c.H * c.dv}}, c.rk, &L.wuv, nullptr) ||
-                    load_stack(st, {{q + "uk", c.H * c.dk}}, c.rk, &L.wuk, nullptr))
-                    return 1;
-                if (need(st, q + "uk", {c.H * c.dk, c.rk}, &t)) return 1;
-                std::vector<float> tr((size_t)c.H * c.rk * c.dk);   // [h][r][d] <- uk[h*dn + d][r]
-                for (int hh = 0; hh < c.H; hh++)
-                    for (int d = 0; d < c.dk; d++)
-                        for (int r = 0; r < c.rk; r++) {
-                            const size_t src = ((size_t)hh * c.dk + d) * c.rk + r;
-                            tr[((size_t)hh * c.rk + r) * c.dk + d] =
-                                t->dtype == "BF16" ? bf16_bits_to_f32(reinterpret_cast<const uint16_t*>(t->data)[src]) : reinterpret_cast<const float*>(t->data)[src];
-                        }
-                if (dalloc(&L.wukT, tr.size()) || upload_host(tr, L.wukT)) return 1;
-                if (dalloc(&L.lcache, (size_t)max_tokens * (c.rk + c.dr)) || dalloc(&L.lcache_op, (size_t)max_tokens * c.rk)) return 1;
-                max_kfull = std::max(max_kfull, c.H * dq); max_vfull = std::max(max_vfull, c.H * c.dv); max_knope = std::max(max_knope, c.H * c.dk);
-                if (c.rot.dims > 0) {
-                    std::vector<double> f;
-                    double mult;
-                    c.rot.freqs(f, mult);
-                    if (this->angle_tables(c.rot.key(), f, mult, &L.rot_cos, &L.rot_sin)) return 1;
-                }
-                max_lat = std::max(max_lat, c.rq);
-                max_qb = std::max(max_qb, c.H * dq);
-                max_qn = std::max(max_qn, c.H * c.dk);
-                max_qa = std::max(max_qa, c.H * (c.rk + c.dr));
-                max_att = std::max(max_att, c.H * c.rk);
-                max_att2 = std::max(max_att2, att_cols);
+                L.lat.c = c.lat;
+                if (this->load_latent(st, q, L.lat)) return 1;
+                L.in_rows = L.lat.in_rows; L.w_in = L.lat.w_in;
             } else {
                 const int nqk = c.G * c.dk, nv = c.H * c.dv, C = 2 * nqk + nv;
                 t = st.find(q + "a1");
@@ -304,7 +254,7 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
             if (load_stack(st, {{q + "o", width}}, att_cols, &L.wo, nullptr)) return 1;
             max_proj = std::max(max_proj, L.in_rows);
             max_H = std::max(max_H, c.H);
-            max_dv = std::max(max_dv, c.kind == MIX_LATENT ? c.rk : c.dv);
+            max_dv = std::max(max_dv, c.dv);
             if (c.moe.on) {
                 const MoeCfg& f = c.moe;
                 if (load_norm(st, p + "norm2", width, L.n2) || load_norm(st, p + "norm2b", width, L.n2b)) return 1;
@@ -331,19 +281,18 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
     int ensure_scratch(size_t rows) override {
         if (rows <= cap) return 0;
         drop_graphs();   // captured launches point into the old scratch
-        for (void* p : {(void*)x, (void*)hn, (void*)d_rows, (void*)h, (void*)lat, (void*)qn, (void*)att, (void*)att2, (void*)xg, (void*)act, (void*)proj,
-                        (void*)qa, (void*)qb, (void*)fa, (void*)fb, (void*)beta, (void*)part, (void*)y, (void*)wts, (void*)eidx, (void*)slot, (void*)row_of,
+        for (void* p : {(void*)x, (void*)hn, (void*)d_rows, (void*)h, (void*)lat, (void*)att, (void*)xg, (void*)act, (void*)proj,
+                        (void*)qa, (void*)fa, (void*)fb, (void*)beta, (void*)part, (void*)y, (void*)wts, (void*)eidx, (void*)slot, (void*)row_of,
                         (void*)grp, (void*)rz})
             dfree(p);
         cap = 0;
         const size_t pairs = rows * std::max(max_top, 1);
         if (dalloc(&x, rows * width) || dalloc(&hn, rows * width) || dalloc(&d_rows, rows) || dalloc(&h, rows * width) ||
-            dalloc(&lat, rows * std::max(max_lat, 1)) || dalloc(&qn, rows * std::max(max_qn, 1)) || dalloc(&att, rows * max_att) ||
-            dalloc(&att2, rows * std::max(max_att2, 1)) || dalloc(&proj, rows * max_proj) || dalloc(&qa, rows * max_qa) ||
-            dalloc(&qb, rows * std::max(max_qb, 1)) || dalloc(&fa, rows * std::max(max_fa, 1)) || dalloc(&fb, rows * std::max(max_fb, 1)) ||
+            dalloc(&lat, rows * std::max(max_lat, 1)) || dalloc(&att, rows * max_att) || dalloc(&proj, rows * max_proj) || dalloc(&qa, rows * max_qa) ||
+            dalloc(&fa, rows * std::max(max_fa, 1)) || dalloc(&fb, rows * std::max(max_fb, 1)) ||
             dalloc(&beta, rows * max_H) || dalloc(&part, (size_t)max_H * MAX_SPLIT * (max_dv + 2)) || dalloc(&xg, pairs * width) ||
             dalloc(&act, pairs * std::max(max_ff, 1)) || dalloc(&y, pairs * width) || dalloc(&wts, pairs) || dalloc(&eidx, pairs) ||
-            dalloc(&slot, pairs) || dalloc(&row_of, pairs) || dalloc(&grp, (size_t)max_E + 1) || dalloc(&rz, rows * std::max(max_E, 1)))
+            dalloc(&slot, pairs) || dalloc(&row_of, pairs) || dalloc(&grp, (size_t)max_E + 1) || dalloc(&rz, rows * std::max(max_E, 1)) || this->ensure_latent_scratch(rows))
             return 1;
         cap = rows;
         return 0;
@@ -402,53 +351,10 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
     }
 
     int mixer_latent(cudaStream_t st, const Layer& L, int T, const PosSrc& ps, uint32_t pos_hint) {
-        const LayerCfg& c = L.c;
-        const int dq = c.dk + c.dr, dl = c.rk + c.dr;
         if (in_proj(st, L, T)) return 1;
-        LatentKvPostParams<AT> kp{};
-        kp.in = proj; kp.ld = L.in_rows; kp.rq = c.rq; kp.rk = c.rk; kp.dr = c.dr; kp.wq = L.dq_norm; kp.wkv = L.dkv_norm; kp.eps = info.eps;
-        kp.rot_dims = c.rot.dims; kp.rot_cos = L.rot_cos; kp.rot_sin = L.rot_sin; kp.cq_out = lat; kp.cache = L.lcache; kp.cache_op = L.lcache_op; kp.ps = ps;
-        if (launch_k("latent_kv_post_kernel", st, pdl_now, latent_kv_post_kernel<AT>, dim3(T), dim3(256), 0, kp)) return 1;
-        EpiParams<AT> eq{}; eq.out = qb; eq.ldo = c.H * dq; eq.scale = 1.0f;
-        if (this->template matmul<EPI_STORE>(st, T, lat, c.rq, L.wuq, nullptr, c.rq, c.H * dq, eq)) return 1;
-        LatentQPostParams<AT> qp{};
-        qp.q = qb; qp.H = c.H; qp.dn = c.dk; qp.dr = c.dr; qp.rk = c.rk; qp.rot_dims = c.rot.dims; qp.rot_cos = L.rot_cos; qp.rot_sin = L.rot_sin;
-        qp.qn_out = qn; qp.qabs = qa; qp.ps = ps;
-        if (c.per_head_ok && (!c.latent_space_ok || (T >= latent_expand_rows && !ps.sp))) {
-            // per-head form: keys and values of positions 0 .. n up-projected from the cached latents, then plain attention.
-            // A graph-replayed step does not know its position on the host: it up-projects to the end of its 64-position
-            // bucket (rows beyond the position are never read by the attention)
-            int n = (int)ps.pos + T;
-            if (ps.sp) n = (int)(pos_hint / ATT_KT + 1 < (uint32_t)MAX_SPLIT ? std::min<uint32_t>(max_tokens, (pos_hint / ATT_KT + 1) * ATT_KT) : max_tokens);
-            if (!kfull && (dalloc(&kfull, (size_t)max_tokens * max_kfull) || dalloc(&vfull, (size_t)max_tokens * max_vfull) || dalloc(&knope, (size_t)max_tokens * max_knope)))
-                return 1;
-            qp.qfull = qa;
-            if (launch_k("latent_q_post_kernel", st, pdl_now, latent_q_post_kernel<AT>, dim3(T, (c.H + 3) / 4), dim3(128), 0, qp)) return 1;
-            EpiParams<AT> ek{}; ek.out = knope; ek.ldo = c.H * c.dk; ek.scale = 1.0f;
-            if (this->template matmul<EPI_STORE>(st, n, L.lcache_op, c.rk, L.wuk, nullptr, c.rk, c.H * c.dk, ek)) return 1;
-            EpiParams<AT> ev2{}; ev2.out = vfull; ev2.ldo = c.H * c.dv; ev2.scale = 1.0f;
-            if (this->template matmul<EPI_STORE>(st, n, L.lcache_op, c.rk, L.wuv, nullptr, c.rk, c.H * c.dv, ev2)) return 1;
-            LatentExpandParams xp{};
-            xp.knope = knope; xp.cache = L.lcache; xp.kfull = kfull; xp.H = c.H; xp.dn = c.dk; xp.dr = c.dr; xp.rk = c.rk;
-            if (launch_k("latent_expand_kernel", st, pdl_now, latent_expand_kernel, dim3(n), dim3(256), 0, xp)) return 1;
-            AttnRowsParams<AT> p{};
-            p.q = qa; p.kcache = kfull; p.vcache = vfull; p.out = att2;
-            p.T = T; p.H = c.H; p.G = c.H; p.dk = dq; p.dv = c.dv; p.scale = c.scale; p.ps = ps; p.k_ld = c.H * dq; p.v_ld = c.H * c.dv;
-            if (this->attention_launch(st, p, part, pos_hint)) return 1;
-            return out_proj(st, T, att2, c.H * c.dv, L.wo, L.n1b);
-        }
-        if (launch_k("latent_q_post_kernel", st, pdl_now, latent_q_post_kernel<AT>, dim3(T, (c.H + 3) / 4), dim3(128), 0, qp)) return 1;
-        // the unrotated query part of head z into the latent space: qa[:, z*dl .. z*dl+rk] = qn[:, z*dn ..] . wukT[z]^T
-        EpiParams<AT> ea{}; ea.out = qa; ea.ldo = c.H * dl; ea.scale = 1.0f;
-        if (this->template matmul_batched<EPI_STORE>(st, T, c.H, qn, c.H * c.dk, c.dk, L.wukT, (long long)c.rk * c.dk, c.dk, c.rk, ea, dl)) return 1;
-        AttnRowsParams<AT> p{};   // one shared key/value head: keys [latent | rotated part], values = the latent
-        p.q = qa; p.kcache = L.lcache; p.vcache = L.lcache; p.out = att;
-        p.T = T; p.H = c.H; p.G = 1; p.dk = dl; p.dv = c.rk; p.scale = c.scale; p.ps = ps; p.k_ld = dl; p.v_ld = dl;
-        if (this->attention_launch(st, p, part, pos_hint)) return 1;
-        // values' up-projection per head: att2[:, z*dv ..] = att[:, z*rk ..] . wuv[z]^T
-        EpiParams<AT> ev{}; ev.act = att2; ev.lda = c.H * c.dv;
-        if (this->template matmul_batched<EPI_ACT>(st, T, c.H, att, c.H * c.rk, c.rk, L.wuv, (long long)c.dv * c.rk, c.rk, c.dv, ev, c.dv)) return 1;
-        return out_proj(st, T, att2, c.H * c.dv, L.wo, L.n1b);
+        const AT* heads = nullptr;
+        if (B::mixer_latent(st, L.lat, T, ps, pos_hint, proj, &heads)) return 1;
+        return out_proj(st, T, heads, L.c.H * L.c.dv, L.wo, L.n1b);
     }
 
     template <int NR, int LPC> int launch_scan(cudaStream_t st, const DeltaScanParams& sp) {
@@ -572,7 +478,7 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
     }
 
     void set_model_option(const char* name, int value) override {
-        if (!strcmp(name, "latent_expand_rows")) latent_expand_rows = std::max(2, value);
+        if (!strcmp(name, "latent_expand_rows")) this->latent_expand_rows = std::max(2, value);
     }
     // test access: what a layer caches per position.  Windowed attention: K and V rows; latent attention: the latent and the
     // rotated key part (as "k" and "v"); delta-rule layers keep no per-position rows.
@@ -585,9 +491,7 @@ template <typename AT, typename WT> class TudatarModel : public DenseModel<AT, W
             GCK(cudaMemcpy(k_out, L.kcache + pos0 * nk, n * nk * 4, cudaMemcpyDeviceToHost));
             GCK(cudaMemcpy(v_out, L.vcache + pos0 * nv, n * nv * 4, cudaMemcpyDeviceToHost));
         } else if (L.c.kind == MIX_LATENT) {
-            const size_t dl = (size_t)L.c.rk + L.c.dr;
-            GCK(cudaMemcpy2D(k_out, (size_t)L.c.rk * 4, L.lcache + pos0 * dl, dl * 4, (size_t)L.c.rk * 4, n, cudaMemcpyDeviceToHost));
-            if (L.c.dr > 0) GCK(cudaMemcpy2D(v_out, (size_t)L.c.dr * 4, L.lcache + pos0 * dl + L.c.rk, dl * 4, (size_t)L.c.dr * 4, n, cudaMemcpyDeviceToHost));
+            return this->read_latent(st, L.lat, pos0, n, k_out, v_out);
         } else { error = "read_kv: a delta-rule layer keeps a state, not rows per position"; return 1; }
         return 0;
     }

@@ -25,6 +25,7 @@ class ModelType(IntEnum):  # src/transformer.rs:50-55
     RUPENEX = 5   # a folder model: state-space / sink-attention layers, dense or routed feed-forward, layer-normed sublayer outputs
     BADEPEL = 6   # a folder model: several residual streams; windowed attention beside gated linear attention, delta-rule layers, dense or routed feed-forward
     BOLAPEL = 7   # a folder model: generalized-delta-rule / chunked sigmoid-attention layers with token shift, norms around every sublayer
+    LUTESUN = 8   # a folder model: windowed latent attention (two forms), dense or routed feed-forward, normed sublayer outputs
 
 
 class QuantType(IntEnum):  # src/quantization.rs:1-6
