@@ -150,6 +150,8 @@ def bench_arch(args):
     --arch bolapel: that architecture (three generalized-delta-rule layers for every chunked sigmoid-attention layer, dense
     feed-forwards) and Tudatar, the closest folder model (a delta rule with a decay per key channel, windowed attention, norms on
     both sides of every sublayer; its chosen experts are as wide as the dense feed-forward), at the same layer shape.
+    --arch lutesun: that architecture (windowed latent attention in its two forms, one dense layer, then routed experts with a shared
+    one) and Tudatar, the closest folder model (latent attention, windowed attention, routed experts), at the same layer shape.
     Prefill: device time (CUDA events on the handle's stream) of one pass over T prompt tokens.  Decode: device time of K
     HBM-resident steps at positions P.. after a P-token prompt, and the same loop end to end through forward_argmax.  Every
     step streams the whole weight set (larger than L2), so no flush is needed between steps."""
@@ -288,7 +290,17 @@ def bench_arch(args):
         folder_model("bolapel", ocfg, md.write_random_bolapel, md.bolapel_matmul_flops_per_token(ocfg) - head_flops,
                      lambda T: md.bolapel_mixer_flops(ocfg, T), md.bolapel_param_bytes(ocfg), kvb,
                      "bf16 weights and operands, f32 accumulation; f32 residual, caches, recurrent states, norms")
-    if args.arch in ("tudatar", "rupenex", "badepel", "bolapel"):
+    if args.arch == "lutesun":
+        top = 4
+        eff = (a.hidden_dim // (top + 1) + 127) // 128 * 128   # chosen experts + the shared one about as wide as Tudatar's chosen experts
+        lcfg = md.lutesun_config(a.dim, a.n_layers, a.vocab_size, heads=a.n_heads, head_dim=a.head_size, rot_dim=64, kv_rank=256, q_rank=768, window=1024,
+                                 ff=a.hidden_dim * 3 // 2, experts=args.arch_experts, identity=2, top=top, groups=3 if (args.arch_experts + 2) % 3 == 0 else 1,
+                                 keep=2 if (args.arch_experts + 2) % 3 == 0 else 1, expert_ff=eff, shared_ff=eff)
+        kvb = sum(min(P + K // 2, L["mixer"]["mask"]["size"]) * (L["mixer"]["kv_rank"] + L["mixer"]["rot_dim"]) * 4 for L in lcfg["layers"])
+        folder_model("lutesun", lcfg, md.write_random_lutesun, md.lutesun_matmul_flops_per_token(lcfg) - head_flops,
+                     lambda T: md.lutesun_mixer_flops(lcfg, T), md.lutesun_param_bytes(lcfg), kvb,
+                     "bf16 weights and operands, f32 accumulation; f32 residual, caches, norms, router")
+    if args.arch in ("tudatar", "rupenex", "badepel", "bolapel", "lutesun"):
         top = 4
         tcfg = md.tudatar_config(a.dim, a.n_layers, a.vocab_size, heads=a.n_heads, kv_heads=a.n_kv_heads, head_dim=a.head_size,
                                  delta_heads=max(1, a.dim // 128), delta_dim=128, experts=args.arch_experts, top=top,
@@ -305,6 +317,24 @@ def bench_arch(args):
         folder_model("tudatar", tcfg, md.write_random_tudatar, md.tudatar_matmul_flops_per_token(tcfg) - head_flops,
                      lambda T: md.tudatar_mixer_flops(tcfg, T), md.tudatar_param_bytes(tcfg), kvb,
                      "bf16 weights and operands, f32 accumulation; f32 caches, recurrent state, norms, router")
+    if args.arch == "lutesun":
+        clocks = sampler.stop()
+        g = out["lutesun"]["decode"]
+        print(json.dumps({
+            "metric": f"decode tok/s Lutesun bf16 at the layer shape of {args.model} (prefill and Tudatar of the same shape in 'arch')",
+            "value": g["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": Wm, "ms_per_step": g["ms_per_step"],
+            "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"model": f"Lutesun {a.n_layers} layers (latent_attention, latent_attention_2, ...; the first with a dense ff {a.hidden_dim * 3 // 2}, the others "
+                                f"{args.arch_experts} experts of ff {eff}, 2 identity, 4 chosen, shared ff {eff}), width {a.dim}, {a.n_heads} heads of "
+                                f"{a.head_size}+64, latent 256+64, query latent 768, window 1024, vocab {a.vocab_size}",
+                       "first_pos": P, "batch": 1, "prefill_lengths": lens,
+                       "l2": "inputs larger than L2 (the active weight set is streamed every step); no flush needed"},
+            "e2e": {"value": g["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 16, "d2h_bytes_per_step": 4,
+                    "api": "forward_argmax(token, pos) -> next token"},
+            "gpu_launches": launches_total[0], "clocks": clocks,
+            "peaks": {"hbm_gb_s": peak_hbm, "hbm_source": peak_src, "bf16_tflops": peak_tf, "bf16_source": tf_src},
+            "arch": out}))
+        return
     if args.arch == "bolapel":
         clocks = sampler.stop()
         g = out["bolapel"]["decode"]
@@ -434,10 +464,10 @@ def main():
     ap.add_argument("--pos", type=int, default=512, help="prompt length / first decode position")
     ap.add_argument("--cpu-steps", type=int, default=16, help="decode steps of the bounded cpu_baseline sample")
     ap.add_argument("--parity-steps", type=int, default=4, help="greedy decode steps replayed on the CPU oracle (0: skip the parity block)")
-    ap.add_argument("--arch-experts", type=int, default=16, help="--arch tudatar / rupenex / badepel / bolapel (its Tudatar): experts per layer (4 are chosen)")
+    ap.add_argument("--arch-experts", type=int, default=16, help="--arch tudatar / rupenex / badepel / lutesun / bolapel (its Tudatar): experts per layer (4 are chosen)")
     ap.add_argument("--arch-streams", type=int, default=4, help="--arch badepel: residual streams per token")
     ap.add_argument("--arch-delta-dim", type=int, default=64, help="--arch bolapel: key and value size of a delta-rule head")
-    ap.add_argument("--arch", default="", choices=["", "genetar", "tudatar", "rupenex", "badepel", "bolapel"],
+    ap.add_argument("--arch", default="", choices=["", "genetar", "tudatar", "rupenex", "badepel", "bolapel", "lutesun"],
                     help="instead of the default workload: prefill and decode throughput of this folder-model architecture (random "
                          "bf16 weights at the layer shape of --model) beside the LMRS Q8_0 Llama of the same shape")
     ap.add_argument("--arch-layers", type=int, default=0, help="--arch: number of layers (0: as many as --model has)")

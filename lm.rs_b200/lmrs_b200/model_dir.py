@@ -1,6 +1,6 @@
 """Model folders (config.json + model.safetensors) for the architectures the library opens by name: a writer, the
-tensor tables of the Genetar, Tudatar, Rupenex, Badepel and Bolapel architectures, and random bf16 weights of a given shape for
-benchmarks and smoke runs.
+tensor tables of the Genetar, Tudatar, Rupenex, Badepel, Bolapel and Lutesun architectures, and random bf16 weights of a given
+shape for benchmarks and smoke runs.
 
 safetensors layout: 8-byte little-endian header length, that many bytes of JSON (name -> dtype, shape, data_offsets
 relative to the end of the header), then the tensor data.
@@ -71,7 +71,7 @@ def genetar_matmul_flops_per_token(cfg):
 
 def write_random(folder, cfg, table, seed=0):
     """random bf16 weights for a tensor table [(name, shape, kind)], streamed to disk tensor by tensor (a full-size model
-    does not have to fit in host memory twice).  kind: matrix (fan-in scaled) | table | ones | scalar | shift | conv | rate |
+    does not have to fit in host memory twice).  kind: matrix (fan-in scaled) | table | head | ones | scalar | shift | conv | rate |
     small | zero | decay | read | write | mixing"""
     os.makedirs(folder, exist_ok=True)
     with open(os.path.join(folder, "config.json"), "w") as f:
@@ -545,3 +545,89 @@ def write_random_bolapel(folder, cfg, seed=0):
     with open(os.path.join(folder, "config.json"), "w") as f:
         json.dump(written_bolapel_config(cfg), f)
     return folder
+
+
+# ---- Lutesun ---------------------------------------------------------------------------------------------------------------
+def lutesun_config(width, n_layers, vocab, *, heads=16, head_dim=64, rot_dim=64, vdim=None, kv_rank=256, q_rank=768, window=1024, ff=8192, dense_layers=1,
+                   experts=16, identity=2, top=4, groups=3, keep=2, router_scale=1.0, expert_ff=2048, shared_ff=2048, embed_scale=1.0, eps=1e-5,
+                   pattern=("latent_attention", "latent_attention_2")):
+    """layers cycle through `pattern`; the first `dense_layers` have a dense feed-forward (ff == 0: none), the others routed experts"""
+    layers = []
+    for i in range(n_layers):
+        kind = pattern[i % len(pattern)]
+        m = {"heads": heads, "dim": head_dim, "rot_dim": rot_dim, "vdim": vdim or head_dim, "kv_rank": kv_rank, "scale": 1.0 / math.sqrt(head_dim + rot_dim),
+             "mask": {"size": window}, "rot": {"base": 500000.0 if kind == "latent_attention" else 10000.0, "dims": rot_dim}}
+        if kind == "latent_attention_2":
+            m["q_rank"] = q_rank
+        if i < dense_layers:
+            f = {"kind": "dense", "ff": ff} if ff else None
+        else:
+            f = {"kind": "moe", "expert": {"ff": expert_ff},
+                 "router": {"experts": experts, "identity": identity, "top": top, "scale": router_scale, "groups": {"count": groups, "keep": keep}}}
+            if shared_ff:
+                f["shared"] = {"ff": shared_ff}
+        layers.append({"type": kind, "mixer": m, "mlp": f})
+    return {"architecture": "Lutesun", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": embed_scale}, "layers": layers}
+
+
+def lutesun_tensors(cfg):
+    """[(name, shape, kind)]; the embedding table is the head as well (kind 'head': gathered by the embedding, streamed by the head)"""
+    w = cfg["width"]
+    out = [("embed", (cfg["vocab"], w), "head")]
+    for i, L in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", L["mixer"], L.get("mlp")
+        q = p + "mix."
+        H, dn, dr, dv, rk = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        out.append((p + "norm1", (w,), "shift"))
+        if L["type"] == "latent_attention":
+            out.append((q + "q", (H * (dn + dr), w), "matrix"))
+        else:
+            out += [(q + "dq", (m["q_rank"], w), "matrix"), (q + "dq.norm", (m["q_rank"],), "ones"), (q + "uq", (H * (dn + dr), m["q_rank"]), "matrix"),
+                    (q + "g", (H, w), "matrix")]
+        out += [(q + "dkv", (rk + dr, w), "matrix"), (q + "dkv.norm", (rk,), "ones"), (q + "uk", (H * dn, rk), "matrix"), (q + "uv", (H * dv, rk), "matrix"),
+                (q + "o", (w, H * dv), "matrix")]
+        if not f:
+            continue
+        out.append((p + "norm2", (w,), "shift"))
+        if f["kind"] == "dense":
+            out += [(p + "mlp.up", (f["ff"], w), "matrix"), (p + "mlp.up.b", (f["ff"],), "shift"), (p + "mlp.down", (w, f["ff"]), "matrix"),
+                    (p + "mlp.down.b", (w,), "shift")]
+            continue
+        r = f["router"]
+        n = r["experts"] + r.get("identity", 0)
+        out += [(p + "mlp.router", (n, w), "matrix"), (p + "mlp.correction", (n,), "zero")]
+        glus = [(f"e{e}", f["expert"]["ff"]) for e in range(r["experts"])]
+        if f.get("shared"):
+            out.append((p + "mlp.shared.sg", (1, w), "matrix"))
+            glus.append(("shared", f["shared"]["ff"]))
+        for e, n in glus:
+            out += [(f"{p}mlp.{e}.gate", (n, w), "matrix"), (f"{p}mlp.{e}.up", (n, w), "matrix"), (f"{p}mlp.{e}.down", (w, n), "matrix")]
+    return out + [("final.norm", (w,), "shift")]
+
+
+def lutesun_param_bytes(cfg, bytes_per_weight=2):
+    """bytes a decode step streams: every matrix of the mixers and dense layers once, the chosen experts (as a uniform router sends
+    them), the embedding table as the head plus one row of it"""
+    total = cfg["width"] * bytes_per_weight
+    for name, shape, _ in lutesun_tensors(cfg):
+        total += int(np.prod(shape)) * bytes_per_weight * _rupenex_active(cfg, name)
+    return int(total)
+
+
+def lutesun_matmul_flops_per_token(cfg):
+    return int(sum(2 * int(np.prod(shape)) * _rupenex_active(cfg, name) for name, shape, kind in lutesun_tensors(cfg) if kind in ("matrix", "head")))
+
+
+def lutesun_mixer_flops(cfg, T):
+    """FLOPs of the attention over a prompt of T tokens, inside the windows, on per-head keys and values"""
+    total = 0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        w = (m.get("mask") or {}).get("size", 0) or T
+        pairs = T * (T + 1) // 2 if T <= w else w * (w + 1) // 2 + (T - w) * w
+        total += 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"]) * pairs
+    return total
+
+
+def write_random_lutesun(folder, cfg, seed=0):
+    return write_random(folder, cfg, lutesun_tensors(cfg), seed)
