@@ -335,9 +335,12 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
     }
 
     template <int RW, int NI, bool SIG> int launch_attn_t(cudaStream_t st, AttnRowsParams<AT> p, int grid_x, int grid_y) {
-        // double-buffered K/V tiles when the head sizes allow 16-byte copies and two CTAs still fit an SM
-        p.nbuf = (p.dk % 4 == 0 && p.dv % 4 == 0 && p.k_ld % 4 == 0 && p.v_ld % 4 == 0 && attn_smem_bytes<RW, NI>(p.dk, p.dv, 2) <= 100 * 1024) ? 2 : 1;
-        const size_t smem = attn_smem_bytes<RW, NI>(p.dk, p.dv, p.nbuf);
+        // K/V tiles by 16-byte copies when the head sizes allow it, double-buffered when two CTAs still fit an SM
+        // (a one-row step has no more CTAs than SMs or little more, so one CTA may take all of an SM's shared memory)
+        const size_t two = attn_smem_bytes<RW, NI>(p.dk, p.dv, 2, p.v_in_k);
+        p.async = p.dk % 4 == 0 && p.dv % 4 == 0 && p.k_ld % 4 == 0 && p.v_ld % 4 == 0;
+        p.nbuf = p.async && two <= (size_t)(p.T == 1 ? 227 : 100) * 1024 ? 2 : 1;
+        const size_t smem = attn_smem_bytes<RW, NI>(p.dk, p.dv, p.nbuf, p.v_in_k);
         if (optin(attn_rows_kernel<AT, RW, NI, SIG>, smem)) return 1;
         return launch_k("attn_rows_kernel", st, pdl_now, attn_rows_kernel<AT, RW, NI, SIG>, dim3(grid_x, grid_y, p.nsplit), dim3(ATT_WARPS * 32), smem, p);
     }
@@ -346,7 +349,15 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         if (ni <= 1) return launch_attn_t<RW, 1, SIG>(st, p, gx, gy);
         if (ni <= 2) return launch_attn_t<RW, 2, SIG>(st, p, gx, gy);
         if (ni <= 4) return launch_attn_t<RW, 4, SIG>(st, p, gx, gy);
-        return launch_attn_t<RW, 8, SIG>(st, p, gx, gy);
+        if constexpr (RW <= 4) {
+            if constexpr (!SIG) {
+                if (ni > 8) return launch_attn_t<RW, 16, SIG>(st, p, gx, gy);   // only a shared latent head is as wide
+            }
+            return launch_attn_t<RW, 8, SIG>(st, p, gx, gy);
+        } else {
+            error = "attention: no wide-tile kernel for this value size";
+            return 1;
+        }
     }
     // attention over T query rows: the caller fills the tensors, head geometry, pitches, scale, soft-cap, window, kept first keys,
     // sink, gates and penalty;
@@ -368,23 +379,32 @@ template <typename AT, typename WT> class DenseModel : public ArchModel {
         const int chunks = (kv_mul + p.HC - 1) / p.HC;
         int rw = 4;
         if (T == 1) rw = p.HC <= 4 ? 1 : (p.HC <= 8 ? 2 : 4);
+        // long portions: eight rows per warp share each read of a key, when two CTAs still fit an SM and every SM gets two
+        else if (p.dv <= 128 && attn_smem_bytes<8, 4>(p.dk, p.dv, 1) <= 112 * 1024 &&
+                 (long long)((T * p.HC + 8 * ATT_WARPS - 1) / (8 * ATT_WARPS)) * p.G * chunks >= 2 * sms)
+            rw = 8;
         p.TQ = std::max(1, rw * ATT_WARPS / p.HC);
         p.nsplit = 1;
         if (T == 1) {   // decode: split the keys so that the GPU has enough CTAs
             p.nsplit = std::max(1, std::min({tiles, MAX_SPLIT, (2 * sms) / std::max(1, p.G * chunks)}));
         }
         const int gx = (T + p.TQ - 1) / p.TQ, gy = p.G * chunks;
-        int rc = rw == 1 ? launch_attn_rw<1, SIG>(st, p, gx, gy) : (rw == 2 ? launch_attn_rw<2, SIG>(st, p, gx, gy) : launch_attn_rw<4, SIG>(st, p, gx, gy));
+        int rc = rw == 1   ? launch_attn_rw<1, SIG>(st, p, gx, gy)
+                 : rw == 2 ? launch_attn_rw<2, SIG>(st, p, gx, gy)
+                 : rw == 4 ? launch_attn_rw<4, SIG>(st, p, gx, gy)
+                           : launch_attn_rw<8, SIG>(st, p, gx, gy);
         if (rc) return rc;
         if (p.nsplit > 1) {
             AttnCombineParams<AT> cp{};
             cp.part = part; cp.gate = p.gate; cp.gate_logits = p.gate_logits; cp.gate_ld = p.gate_ld; cp.out = p.out; cp.rows = T * p.H; cp.H = p.H; cp.dv = p.dv; cp.nsplit = p.nsplit; cp.out_ld = p.out_ld; cp.out_scale = p.out_scale;
-            return launch_k("attn_combine_kernel", st, pdl_now, attn_combine_kernel<AT>, dim3((cp.rows + 3) / 4), dim3(128), 0, cp);
+            return launch_k("attn_combine_kernel", st, pdl_now, attn_combine_kernel<AT>, dim3((cp.rows + 3) / 4, (p.dv + 31) / 32), dim3(128), 0, cp);
         }
         return 0;
     }
     // does the attention kernel have room for these head sizes? (its K, V and probability tiles live in shared memory)
-    static bool attention_fits(int dk, int dv) {
+    // (a shared latent head, whose values are part of its keys, has no V tile and may be twice as wide)
+    static bool attention_fits(int dk, int dv, bool v_in_k = false) {
+        if (v_in_k) return dv <= 512 && (dv <= 256 ? attn_smem_bytes<4, 8>(dk, dv, 1, true) : attn_smem_bytes<4, 16>(dk, dv, 1, true)) <= 227 * 1024;
         return dv <= 256 && attn_smem_bytes<4, 8>(dk, dv, 1) - (size_t)ATT_KT * 32 * 8 * 4 + (size_t)ATT_KT * 32 * ((dv + 31) / 32) * 4 <= 227 * 1024;
     }
     // A decode step has the same launches for every position of a bucket (the key-split count of the attention is the

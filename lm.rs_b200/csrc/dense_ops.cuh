@@ -981,7 +981,9 @@ template <typename AT> struct AttnRowsParams {
     const float* sink;        // [H] or null: exp(sink[head]) is added to the softmax denominator (no key, no value, not scaled)
     const float* gate_logits; int gate_ld;   // or null: output element (t, h, c) is multiplied by sigmoid(gate_logits[t*gate_ld + h*dv + c])
     const float* r1; const float* r2;   // [H] distance penalty r1 * ln(1 + r2 * (i - j)), or null
-    int nbuf;                 // 2: K/V tiles double-buffered with cp.async (needs dk % 4 == 0 and dv % 4 == 0), 1: loaded in place
+    int v_in_k;               // 1: the values are the first dv entries of the K rows (one shared latent head): the K tile is read for both
+    int async;                // 1: K/V tiles come by cp.async (head sizes and pitches in whole 16-byte pieces), 0: by plain loads
+    int nbuf;                 // 2: the tiles are double-buffered (async only), 1: loaded in place
     float scale, softcap;
     int out_ld;               // operand-type elements between consecutive tokens of `out` (H*dv unless the heads are written into a wider row)
     int has_out_scale;        // 1: the output row times out_scale (a mixer that is summed with another one at a fixed weight)
@@ -994,9 +996,11 @@ DN_DEVINL void cp_async16_zfill(void* smem_dst, const void* gsrc, bool valid) { 
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(gsrc), "r"(n) : "memory");
 }
 inline int attn_k_stride(int dk) { const int d4 = (dk + 3) & ~3; return d4 + ((4 - d4 % 32) + 32) % 32; }   // == 4 mod 32
-template <int RW, int NI> inline size_t attn_smem_bytes(int dk, int dv, int nbuf) {
+template <int RW, int NI> inline size_t attn_smem_bytes(int dk, int dv, int nbuf, bool v_in_k = false) {
     const int d4 = (dk + 3) & ~3, R = RW * ATT_WARPS;
-    return ((size_t)R * d4 + (size_t)nbuf * ((size_t)ATT_KT * attn_k_stride(dk) + (size_t)ATT_KT * 32 * NI) + (size_t)R * ATT_KT) * 4;
+    // v_in_k: columns dv .. 32 * NI of the last key row are read (and not used): they reach at most 32 * NI floats behind the tile
+    return ((size_t)R * d4 + (size_t)nbuf * ((size_t)ATT_KT * attn_k_stride(dk) + (v_in_k ? 0 : (size_t)ATT_KT * 32 * NI)) +
+            std::max<size_t>((size_t)R * ATT_KT, v_in_k ? 32 * NI : 0)) * 4;
 }
 // SIG: the weight of a visible key is sigmoid(score * scale + wbias[head]) and the weights are not normalised: no running maximum,
 // no rescaling, the denominator is one (soft-cap, sink and penalty do not apply)
@@ -1010,7 +1014,8 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
     float* Qs = at_sm;                                  // [R][d4]
     float* Ks0 = Qs + (size_t)R * d4;                   // [nbuf][64][ks]
     float* Vs0 = Ks0 + (size_t)p.nbuf * ATT_KT * ks;    // [nbuf][64][DVP]
-    float* Ps = Vs0 + (size_t)p.nbuf * ATT_KT * DVP;    // [R][64]
+    float* Ps = Vs0 + (p.v_in_k ? 0 : (size_t)p.nbuf * ATT_KT * DVP);   // [R][64]
+    const int vs = p.v_in_k ? ks : DVP;                 // floats between the value rows of a tile
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int kv_mul = p.H / p.G;
     const int chunks = (kv_mul + p.HC - 1) / p.HC;
@@ -1059,10 +1064,9 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
         for (int c = 0; c < NI; c++) acc[i][c] = 0.0f;
     }
     const size_t krow = (size_t)p.k_ld, vrow = (size_t)p.v_ld;
-    const bool vec4 = (p.dk & 3) == 0 && (p.dv & 3) == 0 && (p.k_ld & 3) == 0 && (p.v_ld & 3) == 0;
-    const bool async = p.nbuf == 2;
+    const bool async = p.async != 0, two = p.nbuf == 2;
     const float inv_cap2 = p.softcap > 0.0f ? 2.0f / p.softcap : 0.0f;
-    // double-buffered form: the copies of tile i+1 are in flight (cp.async, no registers) while tile i is used
+    // double-buffered form: the copies of tile i+1 are in flight (no registers) while tile i is used
     auto issue_tile = [&](int tile, int buf) {
         const int j0 = tile * ATT_KT;
         float* Kb = Ks0 + (size_t)buf * ATT_KT * ks;
@@ -1073,7 +1077,7 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
             const bool ok = j0 + j < n_keys;
             cp_async16_zfill(Kb + j * ks + d, ok ? p.kcache + (size_t)(j0 + j) * krow + (size_t)g * p.dk + d : p.kcache, ok);
         }
-        for (int e = threadIdx.x; e < ATT_KT * vq; e += blockDim.x) {
+        for (int e = threadIdx.x; !p.v_in_k && e < ATT_KT * vq; e += blockDim.x) {
             const int j = e / vq, c = (e - j * vq) << 2;
             const bool ok = j0 + j < n_keys;
             cp_async16_zfill(Vb + j * DVP + c, ok ? p.vcache + (size_t)(j0 + j) * vrow + (size_t)g * p.dv + c : p.vcache, ok);
@@ -1081,52 +1085,40 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (async) {
-        if (p.dv < DVP)   // value columns beyond vdim are read by the p.V loop: zero them once in both buffers
-            for (int e = threadIdx.x; e < 2 * ATT_KT * (DVP - p.dv); e += blockDim.x) {
+        if (p.dv < DVP && !p.v_in_k)   // value columns beyond vdim are read by the p.V loop: zero them once in every buffer
+            for (int e = threadIdx.x; e < p.nbuf * ATT_KT * (DVP - p.dv); e += blockDim.x) {
                 const int j = e / (DVP - p.dv), c = p.dv + (e - j * (DVP - p.dv));
                 Vs0[(size_t)j * DVP + c] = 0.0f;
             }
-        if (split < n_walk) issue_tile(tile_of(split), 0);
+        if (two && split < n_walk) issue_tile(tile_of(split), 0);
     }
     int buf = 0;
     for (int u = split; u < n_walk; u += p.nsplit) {
         const int tile = tile_of(u);
         const int j0 = tile * ATT_KT;
         float* Ks = Ks0 + (size_t)buf * ATT_KT * ks;
-        float* Vs = Vs0 + (size_t)buf * ATT_KT * DVP;
-        if (async) {
+        float* Vs = p.v_in_k ? Ks : Vs0 + (size_t)buf * ATT_KT * DVP;
+        if (two) {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncthreads();   // this tile has landed for everyone, and everyone is done with the other buffer
             if (u + p.nsplit < n_walk) issue_tile(tile_of(u + p.nsplit), buf ^ 1);
             buf ^= 1;
         } else {
-        __syncthreads();   // previous tile fully consumed (also orders the Qs fill before the first use)
-        if (vec4) {   // head sizes in whole 16-byte pieces: every K and V row of this head starts on a 16-byte boundary
-            const int kq = d4 >> 2;
-            for (int e = threadIdx.x; e < ATT_KT * kq; e += blockDim.x) {
-                const int j = e / kq, d = (e - j * kq) << 2;
-                float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                if (j0 + j < n_keys) v = *reinterpret_cast<const float4*>(p.kcache + (size_t)(j0 + j) * krow + (size_t)g * p.dk + d);
-                *reinterpret_cast<float4*>(Ks + j * ks + d) = v;
+            __syncthreads();   // previous tile fully consumed (also orders the Qs fill before the first use)
+            if (async) {
+                issue_tile(tile, 0);
+                asm volatile("cp.async.wait_group 0;" ::: "memory");
+            } else {
+                for (int e = threadIdx.x; e < ATT_KT * d4; e += blockDim.x) {
+                    const int j = e / d4, d = e - j * d4;
+                    Ks[j * ks + d] = (j0 + j < n_keys && d < p.dk) ? p.kcache[(size_t)(j0 + j) * krow + (size_t)g * p.dk + d] : 0.0f;
+                }
+                for (int e = threadIdx.x; !p.v_in_k && e < ATT_KT * DVP; e += blockDim.x) {
+                    const int j = e / DVP, c = e - j * DVP;
+                    Vs[e] = (j0 + j < n_keys && c < p.dv) ? p.vcache[(size_t)(j0 + j) * vrow + (size_t)g * p.dv + c] : 0.0f;
+                }
             }
-            constexpr int VQ = DVP >> 2;
-            for (int e = threadIdx.x; e < ATT_KT * VQ; e += blockDim.x) {
-                const int j = e / VQ, c = (e - j * VQ) << 2;
-                float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                if (j0 + j < n_keys && c < p.dv) v = *reinterpret_cast<const float4*>(p.vcache + (size_t)(j0 + j) * vrow + (size_t)g * p.dv + c);
-                *reinterpret_cast<float4*>(Vs + j * DVP + c) = v;
-            }
-        } else {
-            for (int e = threadIdx.x; e < ATT_KT * d4; e += blockDim.x) {
-                const int j = e / d4, d = e - j * d4;
-                Ks[j * ks + d] = (j0 + j < n_keys && d < p.dk) ? p.kcache[(size_t)(j0 + j) * krow + (size_t)g * p.dk + d] : 0.0f;
-            }
-            for (int e = threadIdx.x; e < ATT_KT * DVP; e += blockDim.x) {
-                const int j = e / DVP, c = e - j * DVP;
-                Vs[e] = (j0 + j < n_keys && c < p.dv) ? p.vcache[(size_t)(j0 + j) * vrow + (size_t)g * p.dv + c] : 0.0f;
-            }
-        }
-        __syncthreads();
+            __syncthreads();
         }
         float s0[RW], s1[RW];
 #pragma unroll
@@ -1186,7 +1178,7 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
 #pragma unroll
             for (int jj = 0; jj < 4; jj++)
 #pragma unroll
-                for (int c = 0; c < NI; c++) vv[jj][c] = Vs[(size_t)(j + jj) * DVP + c * 32 + lane];
+                for (int c = 0; c < NI; c++) vv[jj][c] = Vs[(size_t)(j + jj) * vs + c * 32 + lane];
 #pragma unroll
             for (int i = 0; i < RW; i++) {
                 const float4 pv = *reinterpret_cast<const float4*>(Ps + (size_t)(warp * RW + i) * ATT_KT + j);
@@ -1219,7 +1211,7 @@ static __global__ void __launch_bounds__(ATT_WARPS * 32) attn_rows_kernel(const 
         }
     }
 }
-// merges the key splits of a row: one warp per (token, head)
+// merges the key splits of a row: one warp per (token, head) and column range (gridDim.y ranges)
 template <typename AT> struct AttnCombineParams {
     const float* part; const float* gate; AT* out;
     const float* gate_logits; int gate_ld;   // per-element sigmoid gates, as in AttnRowsParams
@@ -1242,7 +1234,7 @@ template <typename AT> __global__ void __launch_bounds__(128) attn_combine_kerne
     const float inv = gt * p.out_scale / l;
     const float* gl = p.gate_logits ? p.gate_logits + (size_t)(r / p.H) * p.gate_ld + (size_t)(r % p.H) * p.dv : nullptr;
     AT* dst = p.out + (size_t)(r / p.H) * p.out_ld + (size_t)(r % p.H) * p.dv;
-    for (int c0 = 0; c0 < p.dv; c0 += 32) {
+    for (int c0 = 32 * blockIdx.y; c0 < p.dv; c0 += 32 * gridDim.y) {
         const int c = c0 + lane;
         float a = 0.0f;
 #pragma unroll 8

@@ -54,7 +54,7 @@ template <typename AT, typename WT> class LatentModel : public DenseModel<AT, WT
         if (c.window < 0) { error = where + ": mask.size must not be negative"; return 1; }
         if (c.rot_dims < 0 || c.rot_dims > c.dr || c.rot_dims % 2 != 0) { error = where + ": rot.dims must be even and at most rot_dim"; return 1; }
         // a latent too wide for the attention kernel's tiles is always up-projected to per-head keys and values
-        c.latent_space_ok = D::attention_fits(c.rk + c.dr, c.rk);
+        c.latent_space_ok = D::attention_fits(c.rk + c.dr, c.rk, true);
         c.per_head_ok = D::attention_fits(c.dn + c.dr, c.dv);
         if (!c.latent_space_ok && !c.per_head_ok) { error = where + ": neither kv_rank " + std::to_string(c.rk) + " nor the per-head sizes fit the attention kernel's shared-memory tiles"; return 1; }
         return 0;
@@ -153,7 +153,7 @@ template <typename AT, typename WT> class LatentModel : public DenseModel<AT, WT
         EpiParams<AT> ea{}; ea.out = l_q; ea.ldo = c.H * dl; ea.scale = 1.0f;
         if (this->template matmul_batched<EPI_STORE>(st, T, c.H, l_qn, c.H * c.dn, c.dn, L.wukT, (long long)c.rk * c.dn, c.dn, c.rk, ea, dl)) return 1;
         // one shared key/value head: keys [latent | rotated part], values = the latent
-        p.kcache = L.cache; p.vcache = L.cache; p.out = l_att; p.G = 1; p.dk = dl; p.dv = c.rk; p.k_ld = dl; p.v_ld = dl;
+        p.kcache = L.cache; p.vcache = L.cache; p.out = l_att; p.G = 1; p.dk = dl; p.dv = c.rk; p.k_ld = dl; p.v_ld = dl; p.v_in_k = 1;
         if (this->attention_launch(st, p, l_part, pos_hint)) return 1;
         // values' up-projection per head: out[:, z*dv ..] = att[:, z*rk ..] . wuv[z]^T
         EpiParams<AT> ev{}; ev.act = l_out; ev.lda = c.H * c.dv;

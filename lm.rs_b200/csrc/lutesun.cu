@@ -230,7 +230,7 @@ template <typename AT, typename WT> class LutesunModel : public LatentModel<AT, 
             d.a = act; d.w = L.wdown; d.K = f.ff; d.O = width; d.e = ed; d.bidx = eidx; d.a_bs = f.ff; d.w_bs = (long long)width * f.ff; d.o_bs = width; d.n_mats = f.E;
             if (sh) { d.extra.a = act_sh; d.extra.w = L.sdown; d.extra.K = f.shared_ff; d.extra.O = width; d.extra.out = ysh; }
             if (this->template launch_gemv<EPI_STORE, NORM_NONE>(st, d, f.top + (sh ? 1 : 0))) return 1;
-            return launch_k("moe_combine_resnorm_kernel", st, pdl_now, moe_combine_resnorm_kernel<AT, true>, dim3(1), dim3(one_row_threads()), 0, np);
+            return launch_k("moe_combine_resnorm_kernel", st, pdl_now, moe_combine_resnorm_kernel<AT, true, 4>, dim3(1), dim3(one_row_threads()), 0, np);
         }
         // rows sorted by expert; identity experts sort behind the experts with matrices and take no product
         const int n = T * f.top;
@@ -249,7 +249,8 @@ template <typename AT, typename WT> class LutesunModel : public LatentModel<AT, 
             EpiParams<AT> sd{}; sd.out = ysh; sd.ldo = width; sd.scale = 1.0f;
             if (this->template matmul<EPI_STORE>(st, T, act_sh, f.shared_ff, L.sdown, nullptr, f.shared_ff, width, sd)) return 1;
         }
-        return launch_k("moe_combine_resnorm_kernel", st, pdl_now, moe_combine_resnorm_kernel<AT, false>, dim3(T), dim3(256), 0, np);
+        if (width <= 8 * 256) return launch_k("moe_combine_resnorm_kernel", st, pdl_now, moe_combine_resnorm_kernel<AT, false, 8>, dim3(T), dim3(256), 0, np);
+        return launch_k("moe_combine_resnorm_kernel", st, pdl_now, moe_combine_resnorm_kernel<AT, false, 16>, dim3(T), dim3(256), 0, np);
     }
 
     int run_layers(cudaStream_t st, int T, const PosSrc& ps, uint32_t pos_hint) override {

@@ -85,18 +85,17 @@ template <typename AT> __global__ void __launch_bounds__(256) latent_kv_post_ker
     const int t = blockIdx.x;
     const uint32_t pos = pos_of(p.ps) + (uint32_t)t;
     const float* row = p.in + (size_t)t * p.ld;
-    float ss = 0.0f, inv;
+    const float* kv = row + p.kv_off;
+    float ss = 0.0f, sq = 0.0f, inv;
+    for (int c = threadIdx.x; c < p.rk; c += blockDim.x) ss += kv[c] * kv[c];
     if (p.rq > 0) {
-        for (int c = threadIdx.x; c < p.rq; c += blockDim.x) ss += row[c] * row[c];
-        ss = block_sum(ss, red);
-        inv = 1.0f / sqrtf(ss / (float)p.rq + p.eps);
+        for (int c = threadIdx.x; c < p.rq; c += blockDim.x) sq += row[c] * row[c];
+        sq = block_sum(sq, red);
+        inv = 1.0f / sqrtf(sq / (float)p.rq + p.eps);
         for (int c = threadIdx.x; c < p.rq; c += blockDim.x) from_f(p.cq_out[(size_t)t * p.rq + c], row[c] * inv * p.wq[c]);
     }
     if (p.gate_out)
         for (int h = threadIdx.x; h < p.H; h += blockDim.x) p.gate_out[(size_t)t * p.H + h] = 1.0f / (1.0f + expf(-row[p.gate_off + h]));
-    const float* kv = row + p.kv_off;
-    ss = 0.0f;
-    for (int c = threadIdx.x; c < p.rk; c += blockDim.x) ss += kv[c] * kv[c];
     ss = block_sum(ss, red);
     inv = 1.0f / sqrtf(ss / (float)p.rk + p.eps);
     float* dst = p.cache + (size_t)pos * (p.rk + p.dr);

@@ -252,7 +252,7 @@ struct MoeRow {
     int t;
     float ag;
     template <int CACHE> DN_DEVINL void fill(float (&v)[CACHE]) const {
-        constexpr int KU = CACHE <= 4 ? 4 : 1;   // experts in flight
+        constexpr int KU = CACHE <= 4 ? 4 : (CACHE <= 8 ? 2 : 1);   // experts in flight
 #pragma unroll
         for (int i = 0; i < CACHE; i++) {
             const int c = threadIdx.x + i * blockDim.x;
@@ -286,12 +286,13 @@ template <typename AT> struct MoeCombineResNormParams {
     const float* w; float eps;
     AT* h; int ldh;
 };
-template <typename AT, bool ONE> __global__ void __launch_bounds__(ONE ? 1024 : 256) moe_combine_resnorm_kernel(const MoeCombineResNormParams<AT> p) {
+// CACHE: columns a thread holds (a row of up to CACHE * blockDim.x stays in registers)
+template <typename AT, bool ONE, int CACHE> __global__ void __launch_bounds__(ONE ? 1024 : 256) moe_combine_resnorm_kernel(const MoeCombineResNormParams<AT> p) {
     __shared__ float red[33];
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
-    sandwich_row<AT, ONE ? 4 : 16, ONE>(MoeRow{p.c, t, moe_add_gate(p.c, t)}, p.c.width, p.c.x + (size_t)t * p.c.ldx, p.w, p.eps, red, nullptr, nullptr, nullptr,
+    sandwich_row<AT, CACHE, ONE>(MoeRow{p.c, t, moe_add_gate(p.c, t)}, p.c.width, p.c.x + (size_t)t * p.c.ldx, p.w, p.eps, red, nullptr, nullptr, nullptr,
                                         false, p.h + (size_t)t * p.ldh, nullptr);
 }
 
